@@ -21,11 +21,14 @@ register_architecture("Navalorn", NavalornConfig.from_dict, build_navalorn_spec,
 from .config.torutar import TorutarConfig, build_torutar_spec
 
 register_architecture("Torutar", TorutarConfig.from_dict, build_torutar_spec, replace=True)
+from .config.vavupel import VavupelConfig, build_vavupel_spec
+
+register_architecture("Vavupel", VavupelConfig.from_dict, build_vavupel_spec, replace=True)
 
 from .engine import Engine, Model, StepEntry  # noqa: E402
 from .api import LLM  # noqa: E402
 from .sampling import SamplingParams  # noqa: E402
 
-__all__ = ["ConfigError", "LlamaConfig", "BarovikConfig", "NavalornConfig", "NuzinexConfig", "TorutarConfig", "UnknownArchitectureError", "load_config", "register_architecture",
+__all__ = ["ConfigError", "LlamaConfig", "BarovikConfig", "NavalornConfig", "NuzinexConfig", "TorutarConfig", "VavupelConfig", "UnknownArchitectureError", "load_config", "register_architecture",
            "registered_architectures", "Engine", "Model", "StepEntry", "LLM", "SamplingParams"]
 __version__ = "0.1.0"

@@ -569,6 +569,46 @@ int gi_attn_decode_generic_ex3(void* out, long ldo, float* part_o, float* part_m
                                float scale, int window, int n_splits, int own_tiles, int hdv, float softcap,
                                const float* sinks, int chunk, long v_row_stride, int keep_first, void* stream);
 
+// ---- streams with element-wise tanh norms; embeddings of token pairs (tanh_rows.cu) -------------------------------------
+// v = x + n1(y) per row of d float32 numbers (x or y may be null; rows ldx / ldy apart); n1(u) = tanh(alpha1 u) * w1 + b1, or u
+// (w1 null).  x_out (or null; rows side by side, may be x): v, or `base` (rows ldb apart) in its place.  zero_y: y is zero
+// afterwards.  h (or null; rows side by side, in h_dtype): n2(v) likewise.  `rows` (with neither y nor x_out): the rows of x to
+// read.  settle_of 1 / 2: `settle` describes partial sums pending for x / y (rows of one deferred product's output; they are
+// added to what is read).
+int gi_tanh_rows(const float* x, long ldx, const int* rows, float* y, long ldy, int zero_y, float* x_out, const float* base,
+                 long ldb, float alpha1, const void* w1, const void* b1, float alpha2, const void* w2, const void* b2, int w_dtype,
+                 void* h, int h_dtype, int n_rows, int d, int settle_of, gi_settle_t settle, void* stream);
+// x = cap * tanh(x / cap), float32, in place.
+int gi_softcap_rows(float* x, float cap, long n_values, void* stream);
+// out[t] = table[token_t] * scale + pairs[(prev_t * mul_prev + token_t * mul_cur) mod buckets] (row `buckets` at position 0).
+// prev_t: the token before it in the step, or, for the step's first token of a sequence, state[slot] (int32, rows state_ld
+// apart), which then receives the sequence's last token of the step.  Tokens of one sequence are neighbours in the step.
+int gi_embed_pair(float* out, const void* table, const void* pairs, int w_dtype, const int* tokens, const int* positions,
+                  const int* slots, const int* cu_seqlens, int n_seqs, int* state, long state_ld, int n_tokens, int d, int vocab,
+                  float scale, int buckets, long long mul_prev, long long mul_cur, void* stream);
+
+// ---- additions for attention over a latent in a window, and for linear attention with rotated keys -------------------------
+// gi_latent_prepare and, in the same launch, gi_latent_query_rot (q null: no queries).
+int gi_latent_prepare_q(void* cq, const void* in, int dtype, long ld, const void* wq, const void* wc, int w_dtype, float eps,
+                        const float* table, int rot, const int* positions, const int* slots, const int* block_table, int max_pages,
+                        void* kcache, int n_tokens, int rq, int r, int dr, int write_cache, void* qa, long ldqa, const void* q,
+                        long ldq, int n_heads, int dn, void* stream);
+// gi_attn_latent_tc with a window (0: none), a sink per head (float32, or null) and a gate per token and head (bfloat16 rows
+// ldg apart, or null: a head's output times the gate's sigmoid).
+int gi_attn_latent_tc_ex(void* out, long ldo, float* part_o, float* part_ml, const void* q, long ldq, const void* kcache,
+                         const int* block_table, int max_pages, const int* cu_seqlens, const int* seq_slots, const int* seq_pos0,
+                         const int* seq_lens, int n_seqs, int max_q_len, int n_heads, int dk, int dv, float scale, int n_splits,
+                         int own_tiles, int window, const float* sinks, const void* gate, long ldg, void* stream);
+// gi_attn_combine, each head's result times sigmoid(gate[sequence][head]) (rows ldg apart, in `dtype`).
+int gi_attn_combine_gated(void* out, long ldo, int dtype, const float* part_o, const float* part_ml, int n_seqs, int n_heads, int hd,
+                          int n_splits, const void* gate, long ldg, void* stream);
+// gi_linear_state with constant decays for q and k of `heads` heads whose first 2 * half numbers turn by `table`
+// ([tokens][half] (cos, sin); pairs (i, i + half), or neighbours if `adjacent`), k also times k_scale.
+int gi_linear_state_rot(float* o, const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, int dtype,
+                        const float* decay, const float* table, int half, int adjacent, float k_scale, float* state, long state_ld,
+                        int state_rows, const int* cu_seqlens, const int* seq_slots, int n_seqs, int heads, int K, int V,
+                        int n_tokens, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

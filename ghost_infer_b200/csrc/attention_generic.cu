@@ -313,16 +313,18 @@ attn_decode_kernel(T* __restrict__ out, long ldo, float* __restrict__ part_o, fl
   }
 }
 
-// Merges the slices of one (sequence, head): weights exp(m_s - m), summed in slice order.
+// Merges the slices of one (sequence, head): weights exp(m_s - m), summed in slice order.  `gate` (or null): one number per
+// sequence and head whose sigmoid multiplies the result.
 template <typename T>
 __global__ void attn_combine_kernel(T* __restrict__ out, long ldo, const float* __restrict__ part_o,
-                                    const float* __restrict__ part_ml, int n_heads, int hd, int n_splits) {
+                                    const float* __restrict__ part_ml, int n_heads, int hd, int n_splits, const T* gate, long ldg) {
   // The loads of eight slices are issued together (a slice past the end counts as an empty one): the merge costs
   // a trip or two to the L2 cache, not one per slice.  The arithmetic and its order are those of a plain loop.
   gi::pdl_prologue();
   const int b = blockIdx.y, h = blockIdx.x;
   const size_t p0 = ((size_t)b * n_heads + h) * n_splits;
   const float2* ml = reinterpret_cast<const float2*>(part_ml) + p0;
+  const float open = gate != nullptr ? 1.0f / (1.0f + expf(-gi::ldf(gate + (size_t)b * ldg + h))) : 1.0f;
   if (n_splits <= 8) {
     // the usual case: the maxima, the sums and this thread's values of all slices in one round of loads
     for (int d = threadIdx.x; d < hd; d += blockDim.x) {
@@ -347,7 +349,7 @@ __global__ void attn_combine_kernel(T* __restrict__ out, long ldo, const float* 
           val += o8[j] * w;
         }
       }
-      gi::stf(out + (size_t)b * ldo + (size_t)h * hd + d, tot > 0.f ? val / tot : 0.f);
+      gi::stf(out + (size_t)b * ldo + (size_t)h * hd + d, (tot > 0.f ? val / tot : 0.f) * open);
     }
     return;
   }
@@ -380,7 +382,7 @@ __global__ void attn_combine_kernel(T* __restrict__ out, long ldo, const float* 
         }
       }
     }
-    gi::stf(out + (size_t)b * ldo + (size_t)h * hd + d, tot > 0.f ? val / tot : 0.f);
+    gi::stf(out + (size_t)b * ldo + (size_t)h * hd + d, (tot > 0.f ? val / tot : 0.f) * open);
   }
 }
 
@@ -451,10 +453,15 @@ int pow2_at_least(int v) {
 
 extern "C" int gi_attn_combine(void* out, long ldo, int dtype, const float* part_o, const float* part_ml, int n_seqs,
                                int n_heads, int hd, int n_splits, void* stream) {
+  return gi_attn_combine_gated(out, ldo, dtype, part_o, part_ml, n_seqs, n_heads, hd, n_splits, nullptr, 0, stream);
+}
+
+extern "C" int gi_attn_combine_gated(void* out, long ldo, int dtype, const float* part_o, const float* part_ml, int n_seqs,
+                                     int n_heads, int hd, int n_splits, const void* gate, long ldg, void* stream) {
   dim3 cgrid(n_heads, n_seqs);
   cudaError_t e = cudaSuccess;
   GI_DISPATCH_DTYPE(dtype, T,
-      e = gi::launch(attn_combine_kernel<T>, cgrid, dim3(hd <= 64 ? 64 : (hd <= 128 ? 128 : 256)), 0, (cudaStream_t)stream, (T*)out, ldo, part_o, part_ml, n_heads, hd, n_splits));
+      e = gi::launch(attn_combine_kernel<T>, cgrid, dim3(hd <= 64 ? 64 : (hd <= 128 ? 128 : 256)), 0, (cudaStream_t)stream, (T*)out, ldo, part_o, part_ml, n_heads, hd, n_splits, (const T*)gate, ldg));
   return gi::check(e, "attention combine");
 }
 
@@ -590,7 +597,7 @@ extern "C" int gi_attn_decode_generic_ex3(void* out, long ldo, float* part_o, fl
   if (n_splits > 1) {
     dim3 cgrid(n_heads, n_seqs);
     GI_DISPATCH_DTYPE(dtype, T,
-        (attn_combine_kernel<T><<<cgrid, 64, 0, s>>>((T*)out, ldo, part_o, part_ml, n_heads, hdv, n_splits)));
+        (attn_combine_kernel<T><<<cgrid, 64, 0, s>>>((T*)out, ldo, part_o, part_ml, n_heads, hdv, n_splits, (const T*)nullptr, 0L)));
     return gi::check_launch("attention combine");
   }
   return GI_OK;

@@ -14,6 +14,9 @@
 //  In both, with values wider than 256, a second set of four warps repeats the scores and takes the values' upper half
 //  (a thread cannot hold more than 16 x 256 / 32 sums).
 //  One-token steps cut the context into slices (grid.y); slices are merged by gi_attn_combine.
+// Options, each off at its neutral value: a window (a row at position p sees keys p - window + 1 .. p; a block's walk starts at
+// the tile of the first key any of its rows sees), a learned sink per head (one more term exp(sink) of the softmax's denominator,
+// without key or value; the first slice takes it in), and a gate per token and head (the head's result times the gate's sigmoid).
 // Sizes: dk and dv multiples of 8, dk <= 576, dv <= 512.  Queries' key columns and the tiles' are padded with zeros to a
 // multiple of 16; rows in shared memory are 8 values longer than that, which keeps `ldmatrix` free of bank conflicts.
 #include <math.h>
@@ -27,12 +30,17 @@ namespace {
 constexpr int BQ = 64, BKV = 64;
 constexpr float LOG2E = 1.4426950408889634f, LN2 = 0.6931471805599453f;
 
+__device__ __forceinline__ float head_gate(const __nv_bfloat16* gate, long ldg, int token, int head) {
+  return 1.0f / (1.0f + expf(-gi::ldf(gate + (size_t)token * ldg + head)));
+}
+
 template <int NVT, int DSPLIT, bool KEYS>
 __global__ void __launch_bounds__(128 * DSPLIT)
 attn_latent_mma_kernel(__nv_bfloat16* __restrict__ out, long ldo, float* __restrict__ part_o, float* __restrict__ part_ml,
                        const __nv_bfloat16* q, long ldq, const __nv_bfloat16* kcache, const int* block_table, int max_pages,
                        const int* cu_seqlens, const int* seq_slots, const int* seq_pos0, const int* seq_lens, int n_heads,
-                       float scale, int dk, int dv, int hd, int n_splits, int own_tiles) {
+                       float scale, int dk, int dv, int hd, int n_splits, int own_tiles, int window, const float* __restrict__ sinks,
+                       const __nv_bfloat16* gate, long ldg) {
   constexpr int NT = 128 * DSPLIT;
   constexpr int NS = KEYS ? 2 : BKV / 8;            // key n-tiles a warp forms scores for, per tile
   extern __shared__ __align__(128) unsigned char smem[];
@@ -56,11 +64,12 @@ attn_latent_mma_kernel(__nv_bfloat16* __restrict__ out, long ldo, float* __restr
   const int wr = KEYS ? 0 : (warp & 3), vh = warp >> 2, wk = warp & 3;
   const int rows_here = min(BQ, R - rho0);
   const int p_last = pos0 + (rho0 + rows_here - 1) / n_heads;
-  const int tiles_all = p_last / BKV + 1;
-  int tile_lo = 0, tile_hi = tiles_all;
+  const int k_first = window > 0 ? max(0, pos0 + rho0 / n_heads - window + 1) : 0;     // the first key any row of the block sees
+  const int tile0 = k_first / BKV, tiles_all = p_last / BKV + 1;
+  int tile_lo = tile0, tile_hi = tiles_all;
   if (n_splits > 1) {
-    const int per = own_tiles > 0 ? own_tiles : (tiles_all + n_splits - 1) / n_splits;
-    tile_lo = min(tiles_all, sp * per);
+    const int per = own_tiles > 0 ? own_tiles : (tiles_all - tile0 + n_splits - 1) / n_splits;
+    tile_lo = min(tiles_all, tile0 + sp * per);
     tile_hi = min(tiles_all, tile_lo + per);
   }
   const int ch = hd / 8;
@@ -72,7 +81,7 @@ attn_latent_mma_kernel(__nv_bfloat16* __restrict__ out, long ldo, float* __restr
     __nv_bfloat16* ks = kv_s + (size_t)stage * BKV * ld;
     // a warp takes a row at a time, its lanes the row's 16-byte chunks
     for (int r = warp; r < BKV; r += NT / 32) {
-      const bool seen = kt + r <= p_last;                            // rows nobody here sees, padding columns: zeros
+      const bool seen = kt + r <= p_last && kt + r >= k_first;                            // rows nobody here sees, padding columns: zeros
       for (int c = lane; c < ch; c += 32) {
         const int ok = (seen && c * 8 < dk) ? 16 : 0;
         gi::cp_async_16(gi::smem_u32(ks + r * ld + c * 8), src0 + (ok ? (size_t)r * dk + c * 8 : 0), ok);
@@ -97,6 +106,8 @@ attn_latent_mma_kernel(__nv_bfloat16* __restrict__ out, long ldo, float* __restr
   const bool ok_row[2] = {r_lo < rows_here, r_lo + 8 < rows_here};
   const int p_row[2] = {pos0 + (rho0 + min(r_lo, rows_here - 1)) / n_heads, pos0 + (rho0 + min(r_lo + 8, rows_here - 1)) / n_heads};
   const bool warp_has_rows = wr * 16 < rows_here;
+  const int w_first = window > 0 ? p_row[0] - window + 1 : 0, w_first8 = window > 0 ? p_row[1] - window + 1 : 0;   // first keys of the rows
+  const int p_warp_first_key = window > 0 ? pos0 + (rho0 + min(wr * 16, rows_here - 1)) / n_heads - window + 1 : 0;
   const int p_warp_last = pos0 + (rho0 + min(wr * 16 + 15, rows_here - 1)) / n_heads;
   const float sl2 = scale * LOG2E;
   const int dv16 = (dv + 15) / 16 * 16;
@@ -118,7 +129,7 @@ attn_latent_mma_kernel(__nv_bfloat16* __restrict__ out, long ldo, float* __restr
     const int kt = tile * BKV;
     const __nv_bfloat16* ks_ = kv_s + (size_t)stage * BKV * ld;
     const int key0 = KEYS ? wk * 16 : 0;                         // first key of the tile this warp looks at
-    const bool active = warp_has_rows && kt + key0 <= p_warp_last;
+    const bool active = warp_has_rows && kt + key0 <= p_warp_last && kt + key0 + NS * 8 > p_warp_first_key;
     if (active) {
       float s[NS][4];
 #pragma unroll
@@ -177,7 +188,7 @@ attn_latent_mma_kernel(__nv_bfloat16* __restrict__ out, long ldo, float* __restr
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           const int key = kt + key0 + nt * 8 + 2 * t + (c & 1);
-          const bool ok = ok_row[c >> 1] && key <= p_row[c >> 1];
+          const bool ok = ok_row[c >> 1] && key <= p_row[c >> 1] && key >= ((c >> 1) ? w_first8 : w_first);
           s[nt][c] = ok ? s[nt][c] * sl2 : -INFINITY;
           tmax[c >> 1] = fmaxf(tmax[c >> 1], s[nt][c]);
         }
@@ -240,8 +251,16 @@ attn_latent_mma_kernel(__nv_bfloat16* __restrict__ out, long ldo, float* __restr
       if (row >= rows_here) continue;
       const int rho = rho0 + row;
       const int tokl = rho / n_heads, head = rho % n_heads;
+      float keep = 1.0f;                            // what the sink leaves of the row's sums
+      if (sinks != nullptr && sp == 0) {
+        const float sk = sinks[head] * LOG2E, m_new = fmaxf(m_run[hh], sk);
+        keep = m_run[hh] == -INFINITY ? 0.f : exp2f(m_run[hh] - m_new);
+        l_run[hh] = l_run[hh] * keep + exp2f(sk - m_new);
+        m_run[hh] = m_new;
+      }
       if (n_splits == 1) {
-        const float inv = l_run[hh] > 0.f ? 1.0f / l_run[hh] : 0.f;
+        float inv = l_run[hh] > 0.f ? keep / l_run[hh] : 0.f;
+        if (gate != nullptr) inv *= head_gate(gate, ldg, tok0 + tokl, head);
         __nv_bfloat16* orow = out + (size_t)(tok0 + tokl) * ldo + (size_t)head * dv;
 #pragma unroll
         for (int i = 0; i < NVT; ++i) {
@@ -254,7 +273,7 @@ attn_latent_mma_kernel(__nv_bfloat16* __restrict__ out, long ldo, float* __restr
 #pragma unroll
         for (int i = 0; i < NVT; ++i) {
           const int col = vcol0 + i * 8 + 2 * t;
-          if (col < dv) *reinterpret_cast<float2*>(part_o + pi * dv + col) = make_float2(o[i][hh * 2], o[i][hh * 2 + 1]);
+          if (col < dv) *reinterpret_cast<float2*>(part_o + pi * dv + col) = make_float2(o[i][hh * 2] * keep, o[i][hh * 2 + 1] * keep);
         }
         if (t == 0 && vh == 0) {
           part_ml[pi * 2] = m_run[hh] == -INFINITY ? -INFINITY : m_run[hh] * LN2;
@@ -296,13 +315,19 @@ attn_latent_mma_kernel(__nv_bfloat16* __restrict__ out, long ldo, float* __restr
 #pragma unroll
           for (int w = 0; w < 4; ++w) mx = fmaxf(mx, mm[(half * 4 + w) * 16 + rr]);
           float wgt[4], tot = 0.f;
+          if (sinks != nullptr && sp == 0) {
+            const float sk = sinks[head] * LOG2E;
+            mx = fmaxf(mx, sk);
+            tot = exp2f(sk - mx);
+          }
 #pragma unroll
           for (int w = 0; w < 4; ++w) {
             const float mw = mm[(half * 4 + w) * 16 + rr];
             wgt[w] = (mx == -INFINITY || mw == -INFINITY) ? 0.f : exp2f(mw - mx);
             tot += ml[(half * 4 + w) * 16 + rr] * wgt[w];
           }
-          const float inv = tot > 0.f ? 1.0f / tot : 0.f;
+          float inv = tot > 0.f ? 1.0f / tot : 0.f;
+          if (gate != nullptr && n_splits == 1) inv *= head_gate(gate, ldg, tok0 + tokl, head);
           const int col_end = min(dv, (half + 1) * NVT * 8);
           for (int col = half * NVT * 8 + c0; col < col_end; col += 16) {
             const int cin = col - half * NVT * 8;
@@ -325,7 +350,7 @@ attn_latent_mma_kernel(__nv_bfloat16* __restrict__ out, long ldo, float* __restr
 template <int NVT, int DSPLIT, bool KEYS>
 int launch(dim3 grid, size_t smem, cudaStream_t s, __nv_bfloat16* out, long ldo, float* po, float* pml, const __nv_bfloat16* q, long ldq,
            const __nv_bfloat16* kc, const int* bt, int max_pages, const int* cu, const int* slots, const int* pos0, const int* lens, int H,
-           float scale, int dk, int dv, int hd, int n_splits, int own_tiles) {
+           float scale, int dk, int dv, int hd, int n_splits, int own_tiles, int window, const float* sinks, const __nv_bfloat16* gate, long ldg) {
   auto kern = attn_latent_mma_kernel<NVT, DSPLIT, KEYS>;
   if (KEYS) smem = max(smem, (size_t)4 * DSPLIT * 16 * (NVT * 8 + 8 + 2) * sizeof(float));
   static size_t configured[gi::MAX_DEVICES_SEEN] = {0};
@@ -337,7 +362,7 @@ int launch(dim3 grid, size_t smem, cudaStream_t s, __nv_bfloat16* out, long ldo,
     if (dev >= 0) configured[dev] = smem;
   }
   cudaError_t e = gi::launch(kern, grid, dim3(128 * DSPLIT), smem, s, out, ldo, po, pml, q, ldq, kc, bt, max_pages, cu, slots, pos0,
-                             lens, H, scale, dk, dv, hd, n_splits, own_tiles);
+                             lens, H, scale, dk, dv, hd, n_splits, own_tiles, window, sinks, gate, ldg);
   return gi::check(e, "latent attention (tensor cores)");
 }
 
@@ -348,6 +373,16 @@ extern "C" int gi_attn_latent_tc(void* out, long ldo, float* part_o, float* part
                                  const int* block_table, int max_pages, const int* cu_seqlens, const int* seq_slots,
                                  const int* seq_pos0, const int* seq_lens, int n_seqs, int max_q_len, int n_heads, int dk, int dv,
                                  float scale, int n_splits, int own_tiles, void* stream) {
+  return gi_attn_latent_tc_ex(out, ldo, part_o, part_ml, q, ldq, kcache, block_table, max_pages, cu_seqlens, seq_slots, seq_pos0,
+                              seq_lens, n_seqs, max_q_len, n_heads, dk, dv, scale, n_splits, own_tiles, 0, nullptr, nullptr, 0, stream);
+}
+
+extern "C" int gi_attn_latent_tc_ex(void* out, long ldo, float* part_o, float* part_ml, const void* q, long ldq, const void* kcache,
+                                    const int* block_table, int max_pages, const int* cu_seqlens, const int* seq_slots,
+                                    const int* seq_pos0, const int* seq_lens, int n_seqs, int max_q_len, int n_heads, int dk, int dv,
+                                    float scale, int n_splits, int own_tiles, int window, const float* sinks, const void* gate, long ldg,
+                                    void* stream) {
+  if (window < 0) return gi::fail(GI_ERR_ARG, "latent attention: a window cannot be negative");
   if (n_seqs <= 0 || max_q_len <= 0) return GI_OK;
   if (dk <= 0 || dk > 576 || dk % 8 || dv <= 0 || dv > 512 || dv % 8 || dv > dk)
     return gi::fail(GI_ERR_UNSUPPORTED, "latent attention (tensor cores): rows of %d with values of %d; multiples of 8 up to 576 and 512", dk, dv);
@@ -368,16 +403,16 @@ extern "C" int gi_attn_latent_tc(void* out, long ldo, float* part_o, float* part
 #define GI_LAT(NVT, DS)                                                                                                          \
   rc = keys ? launch<NVT, DS, true>(grid, smem, s, (__nv_bfloat16*)out, ldo, part_o, part_ml, (const __nv_bfloat16*)q, ldq,       \
                                     (const __nv_bfloat16*)kcache, block_table, max_pages, cu_seqlens, seq_slots, seq_pos0, seq_lens, \
-                                    n_heads, scale, dk, dv, hd, n_splits, own_tiles)                                             \
+                                    n_heads, scale, dk, dv, hd, n_splits, own_tiles, window, sinks, (const __nv_bfloat16*)gate, ldg)                                             \
             : launch<NVT, DS, false>(grid, smem, s, (__nv_bfloat16*)out, ldo, part_o, part_ml, (const __nv_bfloat16*)q, ldq,      \
                                      (const __nv_bfloat16*)kcache, block_table, max_pages, cu_seqlens, seq_slots, seq_pos0, seq_lens, \
-                                     n_heads, scale, dk, dv, hd, n_splits, own_tiles)
+                                     n_heads, scale, dk, dv, hd, n_splits, own_tiles, window, sinks, (const __nv_bfloat16*)gate, ldg)
   if (dv16 <= 64) { GI_LAT(8, 1); }
   else if (dv16 <= 128) { GI_LAT(16, 1); }
   else if (dv16 <= 256) { GI_LAT(32, 1); }
   else { GI_LAT(32, 2); }
 #undef GI_LAT
   if (rc != GI_OK) return rc;
-  if (n_splits > 1) return gi_attn_combine(out, ldo, GI_BF16, part_o, part_ml, n_seqs, n_heads, dv, n_splits, stream);
+  if (n_splits > 1) return gi_attn_combine_gated(out, ldo, GI_BF16, part_o, part_ml, n_seqs, n_heads, dv, n_splits, gate, ldg, stream);
   return GI_OK;
 }

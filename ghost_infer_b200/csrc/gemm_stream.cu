@@ -375,7 +375,12 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
             } else if (MODE == GI_SKINNY_STORE_F32) {
               ((float*)out_)[(size_t)m * ldo + f] = v[m];
             } else {
-              ((__nv_bfloat16*)out_)[(size_t)m * ldo + f] = __float2bfloat16_rn(v[m]);
+              float z = v[m];
+              if (MODE == GI_SKINNY_STORE_BF16 && next.act == 2) {      // relu(z)^2
+                z = fmaxf(z, 0.f);
+                z *= z;
+              }
+              ((__nv_bfloat16*)out_)[(size_t)m * ldo + f] = __float2bfloat16_rn(z);
             }
           }
         }
@@ -501,10 +506,10 @@ extern "C" int gi_gemm_stream_bf16_clamped(void* out, const void* A, const void*
 static int gemm_stream_any(void* out, int mode, const void* A, const void* W, float* scratch, int* counters, int n_counters, int M,
                            int N, int K, long lda, long ldw, long ldo, int use_pdl, const void* next_W, int next_N, int next_K,
                            long next_ldw, int next_mode, int units_ahead, float limit, float alpha, void* stream) {
-  const int act = limit > 0.f ? 4 : ((mode & GI_ACT_GELU) ? 1 : 0);
+  const int act = limit > 0.f ? 4 : ((mode & GI_ACT_RELU2) ? 2 : ((mode & GI_ACT_GELU) ? 1 : 0));
   mode &= 0xff;
   next_mode &= 0xff;
-  if (act && mode != GI_SKINNY_SWIGLU) return gi::fail(GI_ERR_ARG, "streamed product: an activation without a gated mode");
+  if (act && mode != (act == 2 ? GI_SKINNY_STORE_BF16 : GI_SKINNY_SWIGLU)) return gi::fail(GI_ERR_ARG, "streamed product: this mode does not take the activation");
   if (M <= 0 || N <= 0) return GI_OK;
   if (M > 64) return gi::fail(GI_ERR_UNSUPPORTED, "streamed product: %d rows of activations, at most 64", M);
   if (K <= 0 || K % 8 != 0 || lda % 8 != 0 || ldw % 8 != 0)

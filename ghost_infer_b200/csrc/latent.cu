@@ -5,7 +5,8 @@
 //  * bias_act:         out = act(in + bias) over rows, and (optionally, in the same launch) residual rows += a bias.
 //  * latent_prepare:   one token's row [query latent | key/value latent | shared rotary key part] of the down product:
 //                      the query latent is RMS-normed for the next product; the key/value latent is RMS-normed and,
-//                      with the rotated key part behind it, written to the token's place in the paged cache.
+//                      with the rotated key part behind it, written to the token's place in the paged cache; where the queries come
+//                      straight out of the same product, their rotary parts as latent_query_rot treats them, in the same launch.
 //  * latent_query_rot: the rotary part of every head's query, rotated, into the rows the attention reads
 //                      ([heads][latent | rotary part]); the latent part of those rows comes from bmm_heads.
 //  * bmm_heads:        out[t, h, :] = W_h a[t, h, :], one small matrix per head (the keys' up-projection folded onto the
@@ -155,14 +156,43 @@ __global__ void bias_act_kernel(T* __restrict__ out, const T* in, long ld_in, co
 }
 
 // ---- the latent's row --------------------------------------------------------------------------------------------
+// The rotary parts of a token's queries (q rows [heads][dn + dr]) into the rows the attention reads (qa rows [heads][r + dr]);
+// q null: the token has none here.
+template <typename T>
+struct LatentQueries {
+  T* qa;
+  long ldqa;
+  const T* q;
+  long ldq;
+  int n_heads, dn;
+};
+template <typename T>
+__device__ __forceinline__ void turn_queries(const LatentQueries<T>& a, int t, const float2* table, int half, int dr, int r) {
+  const int per = dr - half;                       // work items of a head: `half` pairs, then dr - 2 half numbers that pass
+  for (int idx = threadIdx.x; idx < a.n_heads * per; idx += blockDim.x) {
+    const int h = idx / per, i = idx % per;
+    const T* src = a.q + (size_t)t * a.ldq + (size_t)h * (a.dn + dr) + a.dn;
+    T* dst = a.qa + (size_t)t * a.ldqa + (size_t)h * (r + dr) + r;
+    if (i < half) {
+      float x, y;
+      gi::rotate_pair(gi::ldf(src + 2 * i), gi::ldf(src + 2 * i + 1), table[(size_t)t * half + i], &x, &y);
+      gi::stf(dst + 2 * i, x);
+      gi::stf(dst + 2 * i + 1, y);
+    } else {
+      dst[half + i] = src[half + i];
+    }
+  }
+}
+
 template <typename T, typename TW>
 __global__ void __launch_bounds__(128)
 latent_prepare_kernel(T* __restrict__ cq, const T* in, long ld, const TW* __restrict__ wq, const TW* __restrict__ wc, float eps,
                       const float2* table, int half, const int* positions, const int* slots, const int* block_table,
-                      int max_pages, T* kcache, int rq, int r, int dr, int write_cache) {
+                      int max_pages, T* kcache, int rq, int r, int dr, int write_cache, LatentQueries<T> lq) {
   __shared__ float scratch[33];
   gi::pdl_prologue();
   const int t = blockIdx.x;
+  if (lq.q != nullptr) turn_queries(lq, t, table, half, dr, r);
   const T* row = in + (size_t)t * ld;
   // the queries' latent: x / sqrt(mean(x^2) + eps) * w
   if (rq > 0) {
@@ -206,7 +236,7 @@ __global__ void __launch_bounds__(256)
 latent_prepare_vec_kernel(__nv_bfloat16* __restrict__ cq, const __nv_bfloat16* in, long ld, const TW* __restrict__ wq,
                           const TW* __restrict__ wc, float eps, const float2* table, int half, const int* positions,
                           const int* slots, const int* block_table, int max_pages, __nv_bfloat16* kcache, int rq, int r, int dr,
-                          int write_cache) {
+                          int write_cache, LatentQueries<__nv_bfloat16> lq) {
   __shared__ float scratch[33];
   gi::pdl_prologue();
   const int t = blockIdx.x;
@@ -231,6 +261,7 @@ latent_prepare_vec_kernel(__nv_bfloat16* __restrict__ cq, const __nv_bfloat16* i
       if (ci < nq) ssq += ss; else ssc += ss;
     }
   }
+  if (lq.q != nullptr) turn_queries(lq, t, table, half, dr, r);      // while the latents' loads are on their way
   const float rsq = rq > 0 ? 1.0f / sqrtf(gi::block_sum(ssq, scratch) / (float)rq + eps) : 0.f;
   const float rsc = 1.0f / sqrtf(gi::block_sum(ssc, scratch) / (float)r + eps);
   __nv_bfloat16* dst = nullptr;
@@ -267,23 +298,9 @@ latent_prepare_vec_kernel(__nv_bfloat16* __restrict__ cq, const __nv_bfloat16* i
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-latent_query_rot_kernel(T* qa, long ldqa, const T* q, long ldq, const float2* table, int half, int n_heads, int dn, int dr, int r) {
+latent_query_rot_kernel(LatentQueries<T> lq, const float2* table, int half, int dr, int r) {
   gi::pdl_prologue();
-  const int t = blockIdx.x;
-  const int per = dr - half;                       // work items of a head: `half` pairs, then dr - 2 half numbers that pass
-  for (int idx = threadIdx.x; idx < n_heads * per; idx += 256) {
-    const int h = idx / per, i = idx % per;
-    const T* src = q + (size_t)t * ldq + (size_t)h * (dn + dr) + dn;
-    T* dst = qa + (size_t)t * ldqa + (size_t)h * (r + dr) + r;
-    if (i < half) {
-      float a, b;
-      gi::rotate_pair(gi::ldf(src + 2 * i), gi::ldf(src + 2 * i + 1), table[(size_t)t * half + i], &a, &b);
-      gi::stf(dst + 2 * i, a);
-      gi::stf(dst + 2 * i + 1, b);
-    } else {
-      dst[half + i] = src[half + i];
-    }
-  }
+  turn_queries(lq, blockIdx.x, table, half, dr, r);
 }
 
 // ---- one small product per head, CUDA cores ------------------------------------------------------------------------
@@ -558,7 +575,16 @@ extern "C" int gi_latent_prepare(void* cq, const void* in, int dtype, long ld, c
                                  float eps, const float* table, int rot, const int* positions, const int* slots,
                                  const int* block_table, int max_pages, void* kcache, int n_tokens, int rq, int r, int dr,
                                  int write_cache, void* stream) {
+  return gi_latent_prepare_q(cq, in, dtype, ld, wq, wc, w_dtype, eps, table, rot, positions, slots, block_table, max_pages, kcache,
+                             n_tokens, rq, r, dr, write_cache, nullptr, 0, nullptr, 0, 0, 0, stream);
+}
+
+extern "C" int gi_latent_prepare_q(void* cq, const void* in, int dtype, long ld, const void* wq, const void* wc, int w_dtype,
+                                   float eps, const float* table, int rot, const int* positions, const int* slots,
+                                   const int* block_table, int max_pages, void* kcache, int n_tokens, int rq, int r, int dr,
+                                   int write_cache, void* qa, long ldqa, const void* q, long ldq, int n_heads, int dn, void* stream) {
   if (n_tokens <= 0) return GI_OK;
+  if (q != nullptr && (!qa || n_heads <= 0 || dn < 0)) return gi::fail(GI_ERR_ARG, "latent rows: queries without a place or heads");
   if (rq < 0 || r <= 0 || dr < 0 || rot < 0 || rot % 2 != 0 || rot > dr)
     return gi::fail(GI_ERR_ARG, "latent rows: bad sizes (query latent %d, latent %d, rotary part %d of which %d turn)", rq, r, dr, rot);
   if (rot > 0 && table == nullptr) return gi::fail(GI_ERR_ARG, "latent rows: no table of angles");
@@ -569,13 +595,14 @@ extern "C" int gi_latent_prepare(void* cq, const void* in, int dtype, long ld, c
     GI_DISPATCH_DTYPE(w_dtype, TW,
         e = gi::launch(latent_prepare_vec_kernel<TW>, dim3(n_tokens), dim3(256), 0, (cudaStream_t)stream, (__nv_bfloat16*)cq,
                        (const __nv_bfloat16*)in, ld, (const TW*)wq, (const TW*)wc, eps, (const float2*)table, rot / 2, positions, slots,
-                       block_table, max_pages, (__nv_bfloat16*)kcache, rq, r, dr, write_cache));
+                       block_table, max_pages, (__nv_bfloat16*)kcache, rq, r, dr, write_cache,
+                       LatentQueries<__nv_bfloat16>{(__nv_bfloat16*)qa, ldqa, (const __nv_bfloat16*)q, ldq, n_heads, dn}));
     return gi::check(e, "latent rows");
   }
   GI_DISPATCH_DTYPE(dtype, T, GI_DISPATCH_DTYPE(w_dtype, TW,
       e = gi::launch(latent_prepare_kernel<T, TW>, dim3(n_tokens), dim3(128), 0, (cudaStream_t)stream, (T*)cq, (const T*)in, ld,
                      (const TW*)wq, (const TW*)wc, eps, (const float2*)table, rot / 2, positions, slots, block_table, max_pages,
-                     (T*)kcache, rq, r, dr, write_cache)));
+                     (T*)kcache, rq, r, dr, write_cache, LatentQueries<T>{(T*)qa, ldqa, (const T*)q, ldq, n_heads, dn})));
   return gi::check(e, "latent rows");
 }
 
@@ -587,8 +614,8 @@ extern "C" int gi_latent_query_rot(void* qa, long ldqa, const void* q, long ldq,
   if (rot > 0 && table == nullptr) return gi::fail(GI_ERR_ARG, "latent queries: no table of angles");
   cudaError_t e = cudaSuccess;
   GI_DISPATCH_DTYPE(dtype, T,
-      e = gi::launch(latent_query_rot_kernel<T>, dim3(n_tokens), dim3(256), 0, (cudaStream_t)stream, (T*)qa, ldqa,
-                     (const T*)q, ldq, (const float2*)table, rot / 2, n_heads, dn, dr, r));
+      e = gi::launch(latent_query_rot_kernel<T>, dim3(n_tokens), dim3(256), 0, (cudaStream_t)stream,
+                     LatentQueries<T>{(T*)qa, ldqa, (const T*)q, ldq, n_heads, dn}, (const float2*)table, rot / 2, dr, r));
   return gi::check(e, "latent queries");
 }
 

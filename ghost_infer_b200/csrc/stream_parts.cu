@@ -200,7 +200,7 @@ __global__ void gate_mul_kernel(T* __restrict__ out, const T* a, const T* g, lon
   gi::stf(out + i, gi::ldf(a + i) * (act ? z * sigmoid_f(z) : sigmoid_f(z)));
 }
 
-// grid (tokens, groups): 128 threads sum one group
+// grid (tokens, groups): 128 threads sum one group; w null: no weight
 template <typename T, typename TW>
 __global__ void __launch_bounds__(128)
 norm_gate_kernel(T* __restrict__ out, const float* y, const T* g, long ldg, const TW* __restrict__ w, int inner, int gs,
@@ -216,7 +216,45 @@ norm_gate_kernel(T* __restrict__ out, const float* y, const T* g, long ldg, cons
   for (int i = threadIdx.x; i < gs; i += 128) {
     const float z = gi::ldf(g + t * ldg + c0 + i);
     const float gate = act ? z * sigmoid_f(z) : sigmoid_f(z);
-    gi::stf(out + t * inner + c0 + i, yr[i] * rs * gi::ldf(w + (w_per_row ? c0 + i : i)) * gate);
+    gi::stf(out + t * inner + c0 + i, yr[i] * rs * (w != nullptr ? gi::ldf(w + (w_per_row ? c0 + i : i)) : 1.0f) * gate);
+  }
+}
+
+// The same for groups of up to 512 numbers whose parts start on 16-byte boundaries: a warp takes a group, its lanes four
+// neighbouring numbers at a time, kept in registers between the sum and the result.
+constexpr int NG_VEC = 4;
+template <typename T, typename TW>
+__global__ void __launch_bounds__(256)
+norm_gate_warp_kernel(T* __restrict__ out, const float* y, const T* g, long ldg, const TW* __restrict__ w, int inner, int gs,
+                      int w_per_row, int act, float eps, long total_groups) {
+  gi::pdl_prologue();
+  const long grp = (long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (grp >= total_groups) return;
+  const int lane = threadIdx.x & 31, groups = inner / gs;
+  const size_t t = grp / groups;
+  const int c0 = (int)(grp - (long)t * groups) * gs;
+  const float* yr = y + t * inner + c0;
+  float4 v[NG_VEC], z[NG_VEC];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NG_VEC; ++j) {
+    const int i = lane * 4 + 128 * j;
+    v[j] = z[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < gs) { v[j] = gi::ld4(yr + i); z[j] = gi::ld4(g + t * ldg + c0 + i); }
+    ss = fmaf(v[j].x, v[j].x, ss); ss = fmaf(v[j].y, v[j].y, ss); ss = fmaf(v[j].z, v[j].z, ss); ss = fmaf(v[j].w, v[j].w, ss);
+  }
+  const float rs = 1.0f / sqrtf(gi::warp_sum(ss) / (float)gs + eps);
+#pragma unroll
+  for (int j = 0; j < NG_VEC; ++j) {
+    const int i = lane * 4 + 128 * j;
+    if (i >= gs) continue;
+    float4 k = make_float4(sigmoid_f(z[j].x), sigmoid_f(z[j].y), sigmoid_f(z[j].z), sigmoid_f(z[j].w));
+    if (act) { k.x *= z[j].x; k.y *= z[j].y; k.z *= z[j].z; k.w *= z[j].w; }
+    if (w != nullptr) {
+      const float4 ww = gi::ld4(w + (w_per_row ? c0 + i : i));
+      k.x *= ww.x; k.y *= ww.y; k.z *= ww.z; k.w *= ww.w;
+    }
+    gi::st4(out + t * inner + c0 + i, make_float4(v[j].x * rs * k.x, v[j].y * rs * k.y, v[j].z * rs * k.z, v[j].w * rs * k.w));
   }
 }
 
@@ -323,6 +361,14 @@ extern "C" int gi_norm_gate(void* out, int dtype, const float* y, const void* g,
   if (n_rows <= 0) return GI_OK;
   if (inner <= 0 || group <= 0 || inner % group) return gi::fail(GI_ERR_ARG, "norm_gate: %d values do not divide into groups of %d", inner, group);
   cudaError_t e = cudaSuccess;
+  const long total_groups = (long)n_rows * (inner / group);
+  if (group % 4 == 0 && group <= NG_VEC * 128 && ldg % 4 == 0 && (total_groups + 7) / 8 <= 0x7fffffffL &&
+      (((uintptr_t)out | (uintptr_t)y | (uintptr_t)g | (uintptr_t)w) & 15) == 0) {
+    GI_DISPATCH_DTYPE(dtype, T, GI_DISPATCH_DTYPE(w_dtype, TW,
+        e = gi::launch(norm_gate_warp_kernel<T, TW>, dim3((unsigned)((total_groups + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, (T*)out, y,
+                       (const T*)g, ldg, (const TW*)w, inner, group, w_per_row, act, eps, total_groups)));
+    return gi::check(e, "norm_gate");
+  }
   GI_DISPATCH_DTYPE(dtype, T, GI_DISPATCH_DTYPE(w_dtype, TW,
       e = gi::launch(norm_gate_kernel<T, TW>, dim3(n_rows, inner / group), dim3(128), 0, (cudaStream_t)stream, (T*)out, y,
                      (const T*)g, ldg, (const TW*)w, inner, group, w_per_row, act, eps)));

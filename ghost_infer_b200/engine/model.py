@@ -71,6 +71,8 @@ class Model:
         self.embedding = lookup("embedding", spec.embedding.kind)(spec.embedding.params, spec.embedding_prefix)
         en = getattr(spec, "embedding_norm", None)
         self.embedding_norm = None if en is None else lookup("norm", en.kind)(en.params, spec.embedding_norm_prefix)
+        inj = getattr(spec, "injection", None)
+        self.injection = None if inj is None else lookup("injection", inj.kind)(inj.params, spec.injection_prefix)
         self.layers = [Layer(ls, i) for i, ls in enumerate(spec.layers)]
         self.final_norm = lookup("norm", spec.final_norm.kind)(spec.final_norm.params, spec.final_norm_prefix)
         self.head = lookup("head", spec.head.kind)(spec.head.params, spec.head_prefix)
@@ -81,6 +83,8 @@ class Model:
         out = list(self.embedding.weights())
         if self.embedding_norm is not None:
             out.extend(self.embedding_norm.weights())
+        if self.injection is not None:
+            out.extend(self.injection.weights())
         for layer in self.layers:
             out.extend(layer.weights())
         out.extend(self.final_norm.weights())
@@ -105,6 +109,8 @@ class Model:
         self.embedding.bind(tensors, self.rt)
         if self.embedding_norm is not None:
             self.embedding_norm.bind(tensors, self.rt)
+        if self.injection is not None:
+            self.injection.bind(tensors, self.rt)
         for layer in self.layers:
             layer.bind(tensors, self.rt)
         self.final_norm.bind(tensors, self.rt)
@@ -122,6 +128,8 @@ class Model:
                 out.append((i, None, None, e.memory_of, own))
             else:
                 out.append((i, mixer.cache_request(), mixer.state_request(), e.memory_of, own))
+        if getattr(self.embedding, "reads_step", False):       # an embedding's state comes after the scheduled entries'
+            out.append((len(self.spec.schedule), None, self.embedding.state_request(), None, None))
         return out
 
     def new_cache(self, max_tokens: int, max_slots: Optional[int] = None, max_seq_len: Optional[int] = None,

@@ -45,6 +45,7 @@ class StepContext:
         self.logit_rows: Optional[torch.Tensor] = None   # int32 [R] flat token indices
         self.empty_f32: torch.Tensor = None
         self.shared: dict = {}                  # what parts compute once per step and share (e.g. rotary angles)
+        self.next_reader = None                 # the part that reads the stream next after the one running now, where it says what it does
         self.sm_count = 148
         # A step whose launches are recorded once and replayed (a CUDA graph) keeps the plans it was recorded
         # with: id(mixer) -> what the mixer's `decode_plan` returned for the recording's shape.
@@ -136,8 +137,19 @@ class Engine:
             m = layers[e.layer].block.mixer
             if m is not None and all(m is not seen for seen in self._mixers):
                 self._mixers.append(m)
-        parts = [getattr(model, n, None) for n in ("embedding", "embedding_norm", "final_norm", "head")] + [p for layer in layers for p in layer.block.parts()]
+        parts = [getattr(model, n, None) for n in ("embedding", "embedding_norm", "injection", "final_norm", "head")] + [p for layer in layers for p in layer.block.parts()]
         self.plans_on_host = any(getattr(p, "plans_on_host", False) for p in parts)
+        # who reads the stream first at every scheduled entry (the injection where a pass starts), if the block says so;
+        # none over several copies of the stream, which no single pass writes
+        schedule = getattr(model.spec, "schedule", ())
+        self._first_readers = [None] * len(schedule)
+        if not getattr(model.spec, "streams", 0):
+            self._first_readers = [self._block_reader(e) for e in schedule]
+        self._embedding_memory = len(schedule)       # the entry under which the embedding's own state is kept
+
+    def _block_reader(self, entry):
+        block = self.model.layers[entry.layer].block
+        return block.first_reader() if hasattr(block, "first_reader") else None
 
     # ---- host-side checks, before anything is launched (src/model.rs:974-982) -------------------
     def _validate(self, entries: Sequence[StepEntry]) -> None:
@@ -218,15 +230,29 @@ class Engine:
         the wanted rows only (src/model.rs:1173-1188)."""
         from ..kernels import ops
         model = self.model
+        schedule, injection = model.spec.schedule, getattr(model, "injection", None)
+        blocks_read = self._first_readers
+        # who reads the stream right after each entry's turn: the injection where the next entry starts a pass, else the next block
+        reads = [injection if e.inject else r for e, r in zip(schedule, blocks_read)]
+        ctx.next_reader = reads[0] if reads else None
         # the residual stream: a tensor that a deferred product may leave partial sums for (they travel with it)
-        x = model.embedding.forward(ctx.tokens)
+        if getattr(model.embedding, "reads_step", False):
+            x = model.embedding.forward(ctx, self.cache.memory(self._embedding_memory))
+        else:
+            x = model.embedding.forward(ctx.tokens)
         if getattr(model, "embedding_norm", None) is not None:      # the stream stays 32-bit
-            x = model.embedding_norm.forward(x, out_dtype=torch.float32)
+            x = model.embedding_norm.start_stream(x, ctx)
         streams = int(getattr(model.spec, "streams", 0) or 0)
         if streams:                                                  # several copies of the stream, equal at the start
             x = ops.stream_expand(x, streams)
         x = ops.as_carrier(x)
-        for i, e in enumerate(model.spec.schedule):
+        if injection is not None:
+            injection.begin(x, ctx, bool(schedule) and schedule[0].inject)
+        for i, e in enumerate(schedule):
+            if e.inject:
+                ctx.next_reader = blocks_read[i]
+                injection.forward(x, ctx)
+            ctx.next_reader = reads[i + 1] if i + 1 < len(schedule) else None
             model.layers[e.layer].block.forward(x, ctx, self.cache.memory(i))
         if ctx.logit_rows is None:
             ops.drop_pending(x)

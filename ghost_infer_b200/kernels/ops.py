@@ -38,7 +38,7 @@ def _bind():
     if _bound is not None:
         return _bound
     lib = load()
-    P, I, L, F = c_void_p, c_int, c_long, c_float
+    P, I, L, F, LL = c_void_p, c_int, c_long, c_float, ctypes.c_longlong
     sigs = {
         "gi_embed": [P, P, I, P, I, I, I, P],
         "gi_rmsnorm": [P, I, P, P, I, P, I, I, F, P],
@@ -136,6 +136,12 @@ def _bind():
         "gi_moe_route_shares": [P, P, P, P, I, L, P, P, I, I, I, I, I, I, P, F, P],
         "gi_moe_gemm_gate_up_clamped": [P, I, P, L, P, I, L, P, P, I, I, I, I, I, I, F, F, P],
         "gi_attn_prefill_generic_ex3": [P, L, P, L, I, P, P, P, I, P, P, P, I, I, I, I, I, F, I, I, F, P, I, L, I, P],
+        "gi_tanh_rows": [P, L, P, P, L, I, P, P, L, F, P, P, F, P, P, I, P, I, I, I, I, SettleT, P],
+        "gi_softcap_rows": [P, F, L, P],
+        "gi_embed_pair": [P, P, P, I, P, P, P, P, I, P, L, I, I, I, F, I, LL, LL, P],
+        "gi_latent_prepare_q": [P, P, I, L, P, P, I, F, P, I, P, P, P, I, P, I, I, I, I, I, P, L, P, L, I, I, P],
+        "gi_attn_latent_tc_ex": [P, L, P, P, P, L, P, P, I, P, P, P, P, I, I, I, I, I, F, I, I, I, P, P, L, P],
+        "gi_linear_state_rot": [P, P, L, P, L, P, L, I, P, P, I, I, F, P, L, I, P, P, I, I, I, I, I, P],
         "gi_attn_decode_generic_ex3": [P, L, P, P, P, L, I, P, P, P, I, P, P, I, I, I, I, F, I, I, I, I, F, P, I, L, I, P],
     }
     for name, argtypes in sigs.items():
@@ -1752,8 +1758,8 @@ ACT_GELU_ERF = 0x400    # the same: gelu(sum) in its exact (erf) form, no bias
 
 def linear_act(h: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], act: str = "relu2") -> torch.Tensor:
     """act(h W^T + bias) in h's type (`act` "relu2": relu squared; "gelu": the exact (erf) form, without a bias).  A prompt
-    step's product on the tensor cores adds the bias and applies the activation in its epilogue, on the 32-bit sums; other
-    products are followed by `bias_act` or `gelu_rows`."""
+    step's product on the tensor cores adds the bias and applies the activation in its epilogue, on the 32-bit sums, and the
+    streamed product of few rows applies relu2 without a bias in its own; other products are followed by `bias_act` or `gelu_rows`."""
     if act not in ("relu2", "gelu") or (act == "gelu" and bias is not None):
         raise KernelError(f"unknown activation \"{act}\" (relu2, or gelu without a bias)")
     flag = ACT_RELU2 if act == "relu2" else ACT_GELU_ERF
@@ -1768,6 +1774,8 @@ def linear_act(h: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], a
                                              bias.data_ptr() if bias is not None else None, m, n, k, _rows(h, "activations"),
                                              _rows(w, "weights"), n, int(TC_TILE_N), _stream()))
         return out
+    if act == "relu2" and bias is None and skinny_ok(h, w) and USE_STREAM and (w.shape[0] + 127) // 128 <= _STREAM_COUNTERS:
+        return gemm_stream(h, w, SKINNY_STORE_BF16 | ACT_RELU2)       # a few rows: in the streamed product's epilogue
     if act == "gelu":
         return gelu_rows(linear(h, w, out_dtype=h.dtype))
     return bias_act(linear(h, w, out_dtype=h.dtype), bias, act)
@@ -1785,10 +1793,11 @@ def add_row_bias(residual: torch.Tensor, bias: torch.Tensor) -> None:
 
 def latent_prepare(rows: torch.Tensor, w_query_norm: Optional[torch.Tensor], w_latent_norm: torch.Tensor, eps: float,
                    table: Optional[torch.Tensor], rot: int, positions: torch.Tensor, slots: torch.Tensor, memory,
-                   q_rank: int, rank: int, rot_dim: int) -> Optional[torch.Tensor]:
+                   q_rank: int, rank: int, rot_dim: int, queries=None) -> Optional[torch.Tensor]:
     """From rows [query latent (q_rank) | latent (rank) | rotary key part (rot_dim)]: the RMS-normed query latent (returned,
     in the rows' type; None when q_rank is 0), and the token's cache row [RMS-normed latent | key part, its first `rot`
-    numbers turned in neighbouring pairs by `table`] written into `memory`'s pages."""
+    numbers turned in neighbouring pairs by `table`] written into `memory`'s pages.  `queries` = (qa, q, heads, dim): what
+    `latent_query_rot` does with them, in the same launch."""
     lib = _bind()
     _cuda(rows, "latent rows")
     ld = _rows(rows, "latent rows")
@@ -1802,13 +1811,25 @@ def latent_prepare(rows: torch.Tensor, w_query_norm: Optional[torch.Tensor], w_l
         raise KernelError("the latents' norm weights do not fit their sizes")
     cq = torch.empty((n, q_rank), dtype=rows.dtype, device=rows.device) if q_rank else None
     bt = memory.block_table
-    _check(lib, lib.gi_latent_prepare(
+    qa, q, heads, dim = queries if (queries is not None and rot_dim) else (None, None, 0, 0)
+    if q is not None:
+        _latent_query_check(qa, q, heads, dim, rot_dim, rank)
+        if q.dtype != rows.dtype or q.shape[0] != n:
+            raise KernelError("the queries' rows must be as many as the latent rows and of their type")
+    _check(lib, lib.gi_latent_prepare_q(
         cq.data_ptr() if cq is not None else None, rows.data_ptr(), _dt(rows, "latent rows"), ld,
         w_query_norm.data_ptr() if q_rank else None, w_latent_norm.data_ptr(), _dt(w_latent_norm, "norm weights"), float(eps),
         table.data_ptr() if table is not None else None, int(rot), _i32(positions, "positions"), _i32(slots, "slots"),
         _i32(bt, "block table"), bt.shape[1] if bt is not None else 0, memory.k.data_ptr() if write else None, n, q_rank, rank,
-        rot_dim, int(write), _stream()))
+        rot_dim, int(write), qa.data_ptr() if q is not None else None, _rows(qa, "latent queries") if q is not None else 0,
+        q.data_ptr() if q is not None else None, _rows(q, "queries") if q is not None else 0, int(heads), int(dim), _stream()))
     return cq
+
+
+def _latent_query_check(qa: torch.Tensor, q: torch.Tensor, n_heads: int, dim: int, rot_dim: int, rank: int) -> None:
+    _cuda(q, "queries")
+    if q.dtype != qa.dtype or q.shape[1] != n_heads * (dim + rot_dim) or qa.shape[1] != n_heads * (rank + rot_dim) or q.shape[0] != qa.shape[0]:
+        raise KernelError("latent queries: rows of the wrong sizes")
 
 
 def latent_query_rot(qa: torch.Tensor, q: torch.Tensor, table: Optional[torch.Tensor], rot: int, n_heads: int, dim: int,
@@ -1816,9 +1837,7 @@ def latent_query_rot(qa: torch.Tensor, q: torch.Tensor, table: Optional[torch.Te
     """qa[t, h, rank:] = q[t, h, dim:] with its first `rot` numbers turned; q rows [heads][dim + rot_dim], qa rows
     [heads][rank + rot_dim]."""
     lib = _bind()
-    _cuda(q, "queries")
-    if q.dtype != qa.dtype or q.shape[1] != n_heads * (dim + rot_dim) or qa.shape[1] != n_heads * (rank + rot_dim) or q.shape[0] != qa.shape[0]:
-        raise KernelError("latent queries: rows of the wrong sizes")
+    _latent_query_check(qa, q, n_heads, dim, rot_dim, rank)
     _check(lib, lib.gi_latent_query_rot(qa.data_ptr(), _rows(qa, "latent queries"), q.data_ptr(), _rows(q, "queries"),
                                         _dt(q, "queries"), table.data_ptr() if table is not None else None, int(rot), q.shape[0],
                                         n_heads, dim, rot_dim, rank, _stream()))
@@ -1848,25 +1867,33 @@ def attn_latent_tc_ok(dtype: torch.dtype, rank: int, rot_dim: int) -> bool:
                 and rank + rot_dim <= 576 and rank <= 512)
 
 
-def attn_latent_decode_plan(n_seqs: int, max_kv_len: int, sm_count: int, n_heads: int, rank: int, rot_dim: int, dtype: torch.dtype):
+def attn_latent_decode_plan(n_seqs: int, max_kv_len: int, sm_count: int, n_heads: int, rank: int, rot_dim: int, dtype: torch.dtype,
+                            window: Optional[int] = None):
     """(kernel, slices in the launch, tiles per slice) for one-token steps over a latent cache.
     "tensor cores" (bfloat16, sizes the kernel takes): every context cut into equal slices of 64-key tiles, as many as
     fill the GPU once.  "plain": slices of eight 32-key tiles of each sequence's own span, so that a sequence's sums are
-    formed in the same order whatever the step holds."""
+    formed in the same order whatever the step holds.  With a window the span is the tiles that hold its positions."""
     if attn_latent_tc_ok(dtype, rank, rot_dim):
         tiles = (max_kv_len + 63) // 64
+        if window:
+            tiles = min(tiles, (int(window) + 62) // 64 + 1)
         blocks = n_seqs * ((n_heads + 63) // 64)
         # one block per SM (the tiles' ring fills its shared memory): as many slices as make one round of blocks
         return "tensor cores", max(1, min(tiles, sm_count // max(blocks, 1))), 0
     tiles = (max_kv_len + 31) // 32
+    if window:
+        tiles = min(tiles, (int(window) + 30) // 32 + 1)
     return "plain", max(1, (tiles + OWN_LENGTH_TILES - 1) // OWN_LENGTH_TILES), OWN_LENGTH_TILES
 
 
 def attention_latent(qa: torch.Tensor, memory, step, n_heads: int, rank: int, rot_dim: int, scale: float, out: torch.Tensor,
-                     plan=None) -> torch.Tensor:
+                     plan=None, window: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
+                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of all heads over one shared row per position: `memory.k` holds [latent (rank) | rotary key part
     (rot_dim)] per position, a head's query row in `qa` has the same layout (its unrotated part already carried onto the
-    latent), the score is their product times `scale`, and the value is the row's latent: out [tokens, heads * rank]."""
+    latent), the score is their product times `scale`, and the value is the row's latent: out [tokens, heads * rank].
+    `window`: a token sees itself and the window - 1 positions before it; `sinks` float32 [heads]: one more term exp(sink) of
+    the softmax's denominator; `gate` [tokens, heads] in the queries' type: a head's result times its sigmoid."""
     if memory.k is None:
         raise KernelError("attention needs a cache to read from")
     hd = rank + rot_dim
@@ -1881,6 +1908,11 @@ def attention_latent(qa: torch.Tensor, memory, step, n_heads: int, rank: int, ro
     bt = memory.block_table
     tc = (attn_latent_tc_ok(qa.dtype, rank, rot_dim) and qa.stride(0) % 8 == 0 and qa.data_ptr() % 16 == 0
           and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0)
+    window = int(window or 0)
+    if gate is not None and (gate.dtype != qa.dtype or tuple(gate.shape) != (qa.shape[0], n_heads) or not gate.is_cuda):
+        raise KernelError(f"the heads' gates must be [{qa.shape[0]}, {n_heads}] rows of the queries' type")
+    gp, ldg = (gate.data_ptr(), _rows(gate, "gate rows")) if gate is not None else (None, 0)
+    sp = _sinks_ptr(sinks, n_heads)
     if step.is_decode:
         if plan is None:
             plan = attn_latent_decode_plan(step.n_seqs, step.max_kv_len, step.sm_count, n_heads, rank, rot_dim, qa.dtype)
@@ -1893,30 +1925,37 @@ def attention_latent(qa: torch.Tensor, memory, step, n_heads: int, rank: int, ro
             part_ml = torch.empty((step.n_seqs * n_heads * n_splits * 2,), dtype=torch.float32, device=qa.device)
         po, pml = (part_o.data_ptr(), part_ml.data_ptr()) if part_o is not None else (None, None)
         if kind == "tensor cores":
-            _check(lib, lib.gi_attn_latent_tc(
+            _check(lib, lib.gi_attn_latent_tc_ex(
                 out.data_ptr(), _rows(out, "attention output"), po, pml, qa.data_ptr(), _rows(qa, "queries"), memory.k.data_ptr(),
                 _i32(bt, "block table"), bt.shape[1], None, _i32(step.seq_slots, "slots"), None, _i32(step.seq_lens, "lengths"),
-                step.n_seqs, 1, n_heads, hd, rank, float(scale), int(n_splits), int(own_tiles), _stream()), 2 if n_splits > 1 else 1)
+                step.n_seqs, 1, n_heads, hd, rank, float(scale), int(n_splits), int(own_tiles), window, sp, gp, ldg, _stream()),
+                2 if n_splits > 1 else 1)
             return out
-        _check(lib, lib.gi_attn_decode_generic_ex2(
+        _check(lib, lib.gi_attn_decode_generic_ex3(
             out.data_ptr(), _rows(out, "attention output"), po, pml, qa.data_ptr(), _rows(qa, "queries"), _dt(qa, "queries"),
             memory.k.data_ptr(), memory.k.data_ptr(), _i32(bt, "block table"), bt.shape[1],
-            _i32(step.seq_slots, "slots"), _i32(step.seq_lens, "lengths"), step.n_seqs, n_heads, 1, hd, float(scale), 0,
-            int(n_splits), int(own_tiles), rank, 0.0, None, 0, hd, _stream()), 2 if n_splits > 1 else 1)
-        return out
+            _i32(step.seq_slots, "slots"), _i32(step.seq_lens, "lengths"), step.n_seqs, n_heads, 1, hd, float(scale), window,
+            int(n_splits), int(own_tiles), rank, 0.0, sp, 0, hd, 0, _stream()), 2 if n_splits > 1 else 1)
+        return out if gate is None else head_gate_rows(out, gate, n_heads, rank)
     if tc:
-        _check(lib, lib.gi_attn_latent_tc(
+        _check(lib, lib.gi_attn_latent_tc_ex(
             out.data_ptr(), _rows(out, "attention output"), None, None, qa.data_ptr(), _rows(qa, "queries"), memory.k.data_ptr(),
             _i32(bt, "block table"), bt.shape[1], _i32(step.cu_seqlens, "cu_seqlens"), _i32(step.seq_slots, "slots"),
             _i32(step.seq_pos0, "start positions"), None, step.n_seqs, step.max_q_len, n_heads, hd, rank, float(scale), 1, 0,
-            _stream()))
+            window, sp, gp, ldg, _stream()))
         return out
-    _check(lib, lib.gi_attn_prefill_generic_ex2(
+    _check(lib, lib.gi_attn_prefill_generic_ex3(
         out.data_ptr(), _rows(out, "attention output"), qa.data_ptr(), _rows(qa, "queries"), _dt(qa, "queries"),
         memory.k.data_ptr(), memory.k.data_ptr(), _i32(bt, "block table"), bt.shape[1],
         _i32(step.cu_seqlens, "cu_seqlens"), _i32(step.seq_slots, "slots"), _i32(step.seq_pos0, "start positions"), step.n_seqs,
-        step.max_q_len, n_heads, 1, hd, float(scale), 0, rank, 0.0, None, 0, hd, _stream()))
-    return out
+        step.max_q_len, n_heads, 1, hd, float(scale), window, rank, 0.0, sp, 0, hd, 0, _stream()))
+    return out if gate is None else head_gate_rows(out, gate, n_heads, rank)
+
+
+def head_gate_rows(a: torch.Tensor, gate: torch.Tensor, n_heads: int, width: int) -> torch.Tensor:
+    """a[t, h, :] * sigmoid(gate[t, h]) for gates in any activation type (`head_gate` takes them as float32)."""
+    g = gate if gate.dtype == torch.float32 else gate.to(torch.float32)
+    return head_gate(a, g, n_heads, width)
 
 
 # ------------------------------------------------------------------------------------------------
@@ -2027,10 +2066,10 @@ def gate_mul(a: torch.Tensor, gate: torch.Tensor, act: str = "sigmoid") -> torch
     return out
 
 
-def norm_gate(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, group: int, eps: float, act: str,
+def norm_gate(y: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], group: int, eps: float, act: str,
               out_dtype: torch.dtype) -> torch.Tensor:
     """y / sqrt(mean over each group of `group` values (y^2) + eps) * weight * act(gate), the weight per value of a group
-    (`group` values) or of the row."""
+    (`group` values) or of the row; None: no weight."""
     lib = _bind()
     _cuda(y, "recurrence output")
     _cuda(gate, "gate rows")
@@ -2039,12 +2078,13 @@ def norm_gate(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, group: 
         raise KernelError(f"unknown gate \"{act}\" (sigmoid, silu)")
     if y.dtype != torch.float32 or not y.is_contiguous() or gate.dtype != out_dtype or tuple(gate.shape) != (n, inner):
         raise KernelError("the gated norm takes contiguous float32 rows and a gate of the output's type and the rows' shape")
-    if weight.numel() not in (group, inner) or not weight.is_contiguous():
+    if weight is not None and (weight.numel() not in (group, inner) or not weight.is_contiguous()):
         raise KernelError(f"the norm's weight must hold {group} or {inner} values")
     out = torch.empty((n, inner), dtype=out_dtype, device=y.device)
     _check(lib, lib.gi_norm_gate(out.data_ptr(), _dt(out, "normed rows"), y.data_ptr(), gate.data_ptr(), _rows(gate, "gate rows"),
-                                 weight.data_ptr(), _dt(weight, "norm weight"), n, inner, int(group),
-                                 int(weight.numel() == inner and group != inner), 1 if act == "silu" else 0, float(eps), _stream()))
+                                 weight.data_ptr() if weight is not None else None,
+                                 _dt(weight, "norm weight") if weight is not None else F32, n, inner, int(group),
+                                 int(weight is not None and weight.numel() == inner and group != inner), 1 if act == "silu" else 0, float(eps), _stream()))
     return out
 
 
@@ -2405,3 +2445,121 @@ def moe_route_shares(h: torch.Tensor, w_router: torch.Tensor, top: int, correcti
                                         w_router.data_ptr(), None, _dt(w_router, "router weights"), n, width, experts, int(top), 2,
                                         correction.data_ptr() if correction is not None else None, float(weight_scale), _stream()))
     return ids, wts
+
+
+# ---- streams with element-wise tanh norms, embeddings of token pairs, rotated linear attention ---------------------------
+def tanh_rows(x: Optional[torch.Tensor], y: Optional[torch.Tensor], post, pre, out_dtype: Optional[torch.dtype], *,
+              x_out: Optional[torch.Tensor] = None, base: Optional[torch.Tensor] = None, zero_y: bool = False,
+              rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """v = x + post(y); `x_out` receives v (or `base` in its place); returns pre(v) in `out_dtype` (None: nothing).  x, y:
+    float32 rows, either may be None; `post` and `pre`: (alpha, weight, bias) of a norm tanh(alpha u) * weight + bias, or None
+    for the value itself.  `zero_y`: y is zero afterwards.  `rows` (with x alone): the rows to read.  Partial sums that a
+    deferred product left for x or for y are added on the way (and stay in x only where `x_out` writes it back)."""
+    lib = _bind()
+    src = x if x is not None else y
+    if src is None:
+        raise KernelError("tanh rows: nothing to read")
+    d = src.shape[1]
+    for t, what in ((x, "stream rows"), (y, "sublayer rows"), (base, "ready-made rows"), (x_out, "stream rows to write")):
+        if t is None:
+            continue
+        _cuda(t, what, settles=t is x or t is y)
+        if t.dtype != torch.float32 or tuple(t.shape) != tuple(src.shape) or t.stride(1) != 1:
+            raise KernelError(f"{what} must be float32 {tuple(src.shape)}, got {t.dtype} {tuple(t.shape)}")
+    if x_out is not None and not x_out.is_contiguous():
+        raise KernelError("the stream must be written as contiguous rows")
+    wdt = None
+    for norm in (post, pre):
+        if norm is not None:
+            _, w, b = norm
+            if w.numel() != d or b.numel() != d or not w.is_contiguous() or not b.is_contiguous() or w.dtype != b.dtype or (wdt is not None and w.dtype != wdt):
+                raise KernelError(f"the norms' weights and biases must hold {d} contiguous values of one type")
+            wdt = w.dtype
+    settle_of, rec = 0, SettleT(None, None, None, None, 0)
+    for code, t in ((1, x), (2, y)):
+        if t is None or not has_pending(t):
+            continue
+        ok = d % 4 == 0 and not t.__dict__["_gi_pending"][1] and not settle_of and t.is_contiguous() and t.data_ptr() % 16 == 0
+        if code == 1 and rows is None and x_out is None:
+            ok = False                   # the sums would be lost for later readers
+        if ok:
+            settle_of, rec = code, _take_pending(t)[0]
+        else:
+            settle(t)
+    n = rows.numel() if rows is not None else src.shape[0]
+    h = torch.empty((n, d), dtype=out_dtype, device=src.device) if out_dtype is not None else None
+    a1, w1, b1 = post if post is not None else (0.0, None, None)
+    a2, w2, b2 = pre if pre is not None else (0.0, None, None)
+    ptr = lambda t: t.data_ptr() if t is not None else None
+    ld = lambda t: t.stride(0) if t is not None else d
+    _check(lib, lib.gi_tanh_rows(ptr(x), ld(x), _i32(rows, "rows"), ptr(y), ld(y), int(zero_y), ptr(x_out), ptr(base), ld(base),
+                                 float(a1), ptr(w1), ptr(b1), float(a2), ptr(w2), ptr(b2), _DT[wdt] if wdt is not None else F32,
+                                 ptr(h), _dt(h, "normed rows") if h is not None else F32, n, d, settle_of, rec, _stream()))
+    return h
+
+
+def hand_on(x: torch.Tensor, reader, h: torch.Tensor) -> None:
+    """Leaves with the stream `x` what `reader` (its next reader) would compute from it first."""
+    x.__dict__["_gi_handed"] = (reader, h)
+
+
+def take_handed(x: torch.Tensor, reader) -> Optional[torch.Tensor]:
+    """What was left with `x` for `reader`, or None.  Whoever asks, it is gone afterwards: the stream moves on."""
+    left = x.__dict__.pop("_gi_handed", None) if type(x) is Carrier else None
+    return left[1] if left is not None and left[0] is reader else None
+
+
+def softcap_rows(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """x = cap * tanh(x / cap) in place (float32)."""
+    lib = _bind()
+    _cuda(x, "logits")
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise KernelError("the capped values must be contiguous float32")
+    _check(lib, lib.gi_softcap_rows(x.data_ptr(), float(cap), x.numel(), _stream()))
+    return x
+
+
+def embed_pair(table: torch.Tensor, pairs: torch.Tensor, step, state: torch.Tensor, scale: float, mul_prev: int, mul_cur: int) -> torch.Tensor:
+    """float32 rows table[token] * scale + pairs[(previous token * mul_prev + token * mul_cur) mod n], n + 1 the pairs' rows, the
+    last one for a sequence's first token.  `state` int32 [slots + 1, 1]: every sequence's last token, renewed by the step."""
+    lib = _bind()
+    _cuda(table, "embedding table")
+    _cuda(pairs, "pair table")
+    vocab, d = table.shape
+    if not table.is_contiguous() or not pairs.is_contiguous() or pairs.shape[1] != d or pairs.dtype != table.dtype or pairs.shape[0] < 2:
+        raise KernelError("the embedding tables must be contiguous, of one width and one type")
+    if state is None or state.dtype != torch.int32 or state.dim() != 2 or not state.is_contiguous():
+        raise KernelError("the pair embedding needs its per-sequence state: a contiguous int32 matrix")
+    n = step.tokens.numel()
+    out = torch.empty((n, d), dtype=torch.float32, device=table.device)
+    _check(lib, lib.gi_embed_pair(out.data_ptr(), table.data_ptr(), pairs.data_ptr(), _dt(table, "embedding table"),
+                                  _i32(step.tokens, "tokens"), _i32(step.positions, "positions"), _i32(step.token_slots, "slots"),
+                                  _i32(step.cu_seqlens, "cu_seqlens"), step.n_seqs, state.data_ptr(), state.stride(0), n, d, vocab,
+                                  float(scale), pairs.shape[0] - 1, int(mul_prev), int(mul_cur), _stream()))
+    return out
+
+
+def linear_state_rot(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, step, heads: int, key_dim: int, v_dim: int,
+                     decay: torch.Tensor, table: Optional[torch.Tensor], rot: int, adjacent: bool, k_scale: float) -> torch.Tensor:
+    """`linear_state` with constant decays whose queries and keys turn on the way in: the first `rot` numbers of every head by
+    `table` [tokens, rot / 2, 2], keys also times `k_scale`."""
+    lib = _bind()
+    n = q.shape[0]
+    for t, what, width in ((q, "queries", heads * key_dim), (k, "keys", heads * key_dim), (v, "values", heads * v_dim)):
+        _cuda(t, what)
+        if t.dtype != q.dtype or tuple(t.shape) != (n, width) or t.stride(1) != 1:
+            raise KernelError(f"{what} must be [{n}, {width}] rows of the queries' type, got {t.dtype} {tuple(t.shape)}")
+    if state is None or state.dtype != torch.float32 or state.dim() != 2 or not state.is_contiguous() or state.shape[1] < heads * key_dim * v_dim:
+        raise KernelError("the recurrence needs its per-sequence state as a contiguous float32 matrix of at least heads x keys x values")
+    if decay.dtype != torch.float32 or decay.numel() != heads or not decay.is_contiguous() or not decay.is_cuda:
+        raise KernelError(f"the decays must be {heads} float32 values on the device")
+    half = rot // 2
+    if half and (table is None or table.dtype != torch.float32 or tuple(table.shape) != (n, half, 2) or not table.is_contiguous()):
+        raise KernelError(f"the table of angles must be contiguous float32 [{n}, {half}, 2]")
+    o = torch.empty((n, heads * v_dim), dtype=torch.float32, device=q.device)
+    _check(lib, lib.gi_linear_state_rot(
+        o.data_ptr(), q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), _dt(q, "queries"),
+        decay.data_ptr(), table.data_ptr() if half else None, half, int(bool(adjacent)), float(k_scale), state.data_ptr(),
+        state.stride(0), state.shape[0], _i32(step.cu_seqlens, "cu_seqlens"), _i32(step.seq_slots, "slots"), step.n_seqs, heads,
+        key_dim, v_dim, int(n), _stream()))
+    return o

@@ -11,6 +11,12 @@ Interfaces (a new kind of part implements one of them and registers under a name
   `Mixer.decode_plan(n_seqs, max_kv_len, sm_count, kv_lens=None)` says how it cuts the work of one-token steps of that shape
   (anything hashable, or None); a recorded step keeps the plan it was recorded with (`step.plan_of(self)`).
 * `FeedForward.forward(h, residual, step)`: adds its output to `residual` in place.
+  `Norm.start_stream(e, step) -> x`: the stream's first rows from the embedded tokens (a model's norm on its embeddings).
+* `Injection.begin(x0, step, starts)` / `Injection.forward(x, step)`: what happens to the stream right before a pass over
+  looped layers (`starts`: the first pass comes right after the embedding).
+* A part that reads the stream through an operation that whoever writes the stream could do on the way says so with
+  `stream_read(step)` (see `Norm`); the step names the next such reader in `step.next_reader`, and a writer that can do
+  its operation leaves the result with the stream (`ops.hand_on`), where the reader takes it (`ops.take_handed`).
 * `Block.forward(x, step, memory)`: runs one layer's parts in its arrangement.  A block is built from the usual
   four parts (norm, mixer, norm, feed-forward; any may be None) and the extra parts its specification names.
 
@@ -90,9 +96,47 @@ class Part:
         self.rt = rt
 
 
+class StreamRead(NamedTuple):
+    """What the next reader of the stream does first: h = norm(x) (None: x itself) in `dtype`; and what the stream holds
+    afterwards (`base`: rows ready made; None: its own value)."""
+    norm: Optional[Tuple[float, torch.Tensor, torch.Tensor]]
+    dtype: torch.dtype
+    base: Optional[torch.Tensor] = None
+
+
 class Norm(Part):
     def forward(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         raise NotImplementedError
+
+    def start_stream(self, e: torch.Tensor, step) -> torch.Tensor:
+        """The embedded tokens, normed: the stream's first rows (32-bit)."""
+        return self.forward(e, out_dtype=torch.float32)
+
+    def stream_read(self, step) -> Optional[StreamRead]:
+        """Element-wise norms can run inside the pass that writes the stream: what that pass has to know.  None: they cannot."""
+        return None
+
+
+class Embedding(Part):
+    """A table of token vectors.  `reads_step`: `forward(step, memory)` gets the whole step and the embedding's own memory
+    (`state_request`) instead of the token ids alone."""
+    reads_step = False
+
+    def state_request(self) -> Optional[StateRequest]:
+        return None
+
+
+class Injection(Part):
+    """What the stream passes through right before every pass over a model's looped layers."""
+
+    def begin(self, x0: torch.Tensor, step, starts: bool) -> None:
+        raise NotImplementedError
+
+    def forward(self, x: torch.Tensor, step) -> None:
+        raise NotImplementedError
+
+    def stream_read(self, step) -> Optional[StreamRead]:
+        return None
 
 
 class PositionEncoding(Part):
@@ -150,6 +194,10 @@ class Block:
 
     def state_request(self) -> Optional[StateRequest]:
         """Fixed-size memory per sequence that the arrangement itself wants (`memory.block_state`); None: nothing."""
+        return None
+
+    def first_reader(self) -> Optional[Part]:
+        """The part that reads the stream first, where that is all the block does with it until then; None: not said."""
         return None
 
     def parts(self):

@@ -13,6 +13,9 @@ class PreNormResidual(Block):
     """x += mixer(norm(x)); x += ffn(norm(x)), the residual stream x kept in 32-bit
     (src/model.rs:996-1147; the reference's stream is f32 too, src/model.rs:704-705)."""
 
+    def first_reader(self):
+        return self.mixer_norm
+
     def forward(self, x, step, memory) -> None:
         # The last product of the mixer and of the feed-forward adds into x; in a decode step it may leave
         # partial sums pending for the norm that reads x next (a norm that cannot add them has them settled first).
@@ -58,3 +61,38 @@ class ResidualPostNorm(Block):
             part.forward(h, x, step)
             if low and i + 1 < len(after):
                 h = ops.cast_rows(x, dt)
+
+
+@register("block", "sandwich_residual")
+class SandwichResidual(Block):
+    """x += n1b(mixer(n1(x))); x += n2b(ffn(n2(x))): a norm before every sublayer and one on what it gives back
+    (`extra["mixer_post"]`, `extra["ffn_post"]`).  Stream, norms and sums are 32-bit.  A sublayer's last product may leave partial
+    sums pending in its rows; a norm whose `join` can do so adds them, joins the rows to the stream and does the first operation
+    of whoever reads the stream next, in one pass; other norms do these one after the other."""
+
+    def first_reader(self):
+        return self.mixer_norm
+
+    def _sublayer(self, x, step, pre, post, run, reader) -> None:
+        if x.is_cuda and not getattr(pre, "settles_pending", False):
+            ops.settle(x)
+        h = pre.forward(x)
+        # the rows a sublayer adds into: zeroed once a step, and again by every join for the next sublayer
+        key = ("sublayer rows", tuple(x.shape))
+        y = step.shared.get(key)
+        if y is None:
+            y = step.shared[key] = ops.as_carrier(torch.zeros(x.shape, dtype=torch.float32, device=x.device))
+        with ops.defer_into(y):
+            run(h, y)
+        if hasattr(post, "join"):
+            post.join(x, y, reader, step, zero_y=True)
+        else:
+            ops.settle(y)
+            post.add_normed(x, y, zero_y=True)
+
+    def forward(self, x, step, memory) -> None:
+        last = step.next_reader
+        self._sublayer(x, step, self.mixer_norm, self.extra["mixer_post"], lambda h, y: self.mixer.forward(h, y, step, memory),
+                       self.ffn_norm if self.ffn is not None else last)
+        if self.ffn is not None:
+            self._sublayer(x, step, self.ffn_norm, self.extra["ffn_post"], lambda h, y: self.ffn.forward(h, y, step), last)

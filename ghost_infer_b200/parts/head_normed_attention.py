@@ -30,8 +30,7 @@ import torch
 from ..cache.sequence_cache import CacheRequest
 from ..kernels import ops
 from .base import Mixer, WeightSpec
-from .linear import linear
-from .linear_state import _stack
+from .linear import linear, stack_rows
 from .registry import register
 from .rope import Rotary
 
@@ -115,7 +114,7 @@ class HeadNormedAttention(Mixer):
             mats += [rt.place(tensors[n["k"]]), rt.place(tensors[n["v"]])]
         if self.head_gate:
             mats.append(rt.place(tensors[n["g"]]))
-        self.w_in = _stack(mats, rt)          # one product with 32-bit results: [q | k | v | one gate per head]
+        self.w_in = stack_rows(mats)              # one product with 32-bit results: [q | k | v | one gate per head]
         del mats
         self.w_o = rt.place(tensors[n["o"]])
         # what enters a norm or the softmax is 32-bit whatever the file stores; biases join the projection's 32-bit sums

@@ -1,4 +1,4 @@
-"""Mixers that carry a matrix of state per head from token to token: a gated delta rule and decayed linear attention.
+"""Mixers that carry a matrix of state per head from token to token: a gated delta rule, decayed linear attention, retention.
 
 Both walk, per head, S (a key_dim x v_dim matrix of 32-bit numbers, zero when a sequence starts):
 
@@ -15,6 +15,11 @@ silu(Wg h); residual += Wo (...).  Per sequence: S and the convolution's last `c
 constant per head (`decay`); the concatenated heads are RMS-normed together (weight of heads * v_dim, eps), multiplied by
 sigmoid(Wg h), and projected: residual += Wo (...).  Per sequence: S.
 
+"retention": q = Wq h, k = Wk h (heads of key_dim), v = Wv h (heads of v_dim), no activation; the position encoding
+(`params["position"]`, a rotary part, or None) turns q and k, and k is multiplied by key_dim^(-1/2); g is a constant per head
+(`decay`); each head's o is divided by its root mean square over v_dim (eps, no weight), the heads side by side are multiplied
+by silu(Wg h), and projected: residual += Wo (...).  Per sequence: S.
+
 The recurrence, decays, gates of the recurrence, unit norms and output norms are 32-bit in both precisions.
 Tensor names: prefix + `base` + {q, q.conv, k, k.conv, v, v.conv, b, a, A_log, dt_bias, norm, g, o} (`base` "mix.").
 """
@@ -27,19 +32,8 @@ import torch
 from ..cache.sequence_cache import StateRequest
 from ..kernels import ops
 from .base import Mixer, WeightSpec
-from .linear import linear
-from .registry import register
-
-
-def _stack(mats, rt) -> torch.Tensor:
-    """Matrices stacked by rows for one product, padded with zero rows to a multiple of 8 rows."""
-    if len({m.dtype for m in mats}) > 1:
-        mats = [m.to(torch.float32) for m in mats]
-    w = torch.cat(mats, dim=0)
-    pad = (-w.shape[0]) % 8
-    if pad:
-        w = torch.cat([w, torch.zeros((pad, w.shape[1]), dtype=w.dtype, device=w.device)], dim=0)
-    return w.contiguous()
+from .linear import linear, stack_rows
+from .registry import lookup, register
 
 
 @register("mixer", "gated_delta_rule")
@@ -82,7 +76,7 @@ class GatedDeltaRule(Mixer):
         super().bind(tensors, rt)
         n = self.names
         # one product: [q | k | v | gate | beta | decay]; the convolved channels come first
-        self.w_in = _stack([rt.place(tensors[n[k]]) for k in ("q", "k", "v", "g", "b", "a")], rt)
+        self.w_in = stack_rows([rt.place(tensors[n[k]]) for k in ("q", "k", "v", "g", "b", "a")])
         self.w_o = rt.place(tensors[n["o"]])
         cw = [rt.place(tensors[n[k]]) for k in ("q.conv", "k.conv", "v.conv")]
         if len({c.dtype for c in cw}) > 1:
@@ -140,7 +134,7 @@ class DecayedLinearAttention(Mixer):
     def bind(self, tensors, rt) -> None:
         super().bind(tensors, rt)
         n = self.names
-        self.w_in = _stack([rt.place(tensors[n[k]]) for k in ("q", "k", "v", "g")], rt)
+        self.w_in = stack_rows([rt.place(tensors[n[k]]) for k in ("q", "k", "v", "g")])
         self.w_o = rt.place(tensors[n["o"]])
         self.norm_w = tensors[n["norm"]].to(device=rt.device, dtype=torch.float32).contiguous()
         self.decay_dev = torch.tensor(self.decay, dtype=torch.float64).to(device=rt.device, dtype=torch.float32)
@@ -156,5 +150,58 @@ class DecayedLinearAttention(Mixer):
                                  self.heads, self.key_dim, self.v_dim, self.decay_dev, in_act=True)
         with ops.bucket("gated norm"):
             y = ops.norm_gate(o, proj[:, 2 * qk + vw:2 * qk + 2 * vw], self.norm_w, vw, self.eps, "sigmoid", self.rt.dtype)
+        with ops.bucket("out matmul"):
+            linear(y, self.w_o, out=residual, accumulate=True)
+
+
+@register("mixer", "retention")
+class Retention(Mixer):
+    def __init__(self, params, prefix=""):
+        super().__init__(params, prefix)
+        self.hidden = int(params["hidden_size"])
+        self.heads = int(params["heads"])
+        self.key_dim = int(params["key_dim"])
+        self.v_dim = int(params["v_dim"])
+        self.eps = float(params["eps"])
+        self.decay = tuple(float(g) for g in params["decay"])
+        if len(self.decay) != self.heads:
+            raise ValueError(f"{len(self.decay)} decays for {self.heads} heads")
+        pos = params.get("position")
+        self.position = lookup("position", pos.kind)(pos.params, prefix) if pos is not None else None
+        self.rot = int(self.position.rotary_dim) if self.position is not None else 0
+        self.adjacent = self.position is not None and self.position.pairing == "adjacent"
+        self.qk_width, self.v_width = self.heads * self.key_dim, self.heads * self.v_dim
+        base = str(params.get("base", "mix."))
+        self.names = {k: self.tensor_name(k, base + k) for k in ("q", "k", "v", "g", "o")}
+
+    def weights(self) -> List[WeightSpec]:
+        n, d = self.names, self.hidden
+        return [WeightSpec(n["q"], (self.qk_width, d)), WeightSpec(n["k"], (self.qk_width, d)), WeightSpec(n["v"], (self.v_width, d)),
+                WeightSpec(n["g"], (self.v_width, d)), WeightSpec(n["o"], (d, self.v_width))]
+
+    def state_request(self) -> Optional[StateRequest]:
+        return StateRequest((self.heads * self.key_dim * self.v_dim,), torch.float32)
+
+    def bind(self, tensors, rt) -> None:
+        super().bind(tensors, rt)
+        n = self.names
+        self.w_in = stack_rows([rt.place(tensors[n[k]]) for k in ("q", "k", "v", "g")])
+        self.w_o = rt.place(tensors[n["o"]])
+        self.decay_dev = torch.tensor(self.decay, dtype=torch.float64).to(device=rt.device, dtype=torch.float32)
+        if self.position is not None:
+            self.position.bind(tensors, rt)
+
+    def forward(self, h, residual, step, memory) -> None:
+        if memory.state is None:
+            raise RuntimeError("retention was given no per-sequence state")
+        qk, vw = self.qk_width, self.v_width
+        with ops.bucket("qkv matmul"):
+            proj = linear(h, self.w_in, out_dtype=self.rt.dtype)
+        with ops.bucket("scan"):
+            table = self.position.table(step) if self.position is not None else None
+            o = ops.linear_state_rot(proj[:, :qk], proj[:, qk:2 * qk], proj[:, 2 * qk:2 * qk + vw], memory.state, step, self.heads,
+                                     self.key_dim, self.v_dim, self.decay_dev, table, self.rot, self.adjacent, self.key_dim ** -0.5)
+        with ops.bucket("gated norm"):
+            y = ops.norm_gate(o, proj[:, 2 * qk + vw:2 * qk + 2 * vw], None, self.v_dim, self.eps, "silu", self.rt.dtype)
         with ops.bucket("out matmul"):
             linear(y, self.w_o, out=residual, accumulate=True)

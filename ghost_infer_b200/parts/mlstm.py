@@ -24,8 +24,7 @@ import torch
 from ..cache.sequence_cache import StateRequest
 from ..kernels import ops
 from .base import Mixer, WeightSpec
-from .linear import linear
-from .linear_state import _stack
+from .linear import linear, stack_rows
 from .registry import register
 
 _KEYS = ("q", "k", "v", "i", "i.b", "f", "f.b", "g", "norm", "o")
@@ -62,7 +61,7 @@ class MLstm(Mixer):
         super().bind(tensors, rt)
         n = self.names
         # one product with 32-bit results: [q | k | v | gate | i | f]
-        self.w_in = _stack([rt.place(tensors[n[k]]) for k in ("q", "k", "v", "g", "i", "f")], rt)
+        self.w_in = stack_rows([rt.place(tensors[n[k]]) for k in ("q", "k", "v", "g", "i", "f")])
         self.w_o = rt.place(tensors[n["o"]])
         f32 = lambda name: tensors[name].to(device=rt.device, dtype=torch.float32).contiguous()
         self.b_i, self.b_f, self.norm_w = f32(n["i.b"]), f32(n["f.b"]), f32(n["norm"])

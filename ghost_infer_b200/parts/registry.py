@@ -3,7 +3,7 @@ from __future__ import annotations
 
 from typing import Callable, Dict
 
-_KINDS = ("norm", "position", "mixer", "feed_forward", "block", "embedding", "head")
+_KINDS = ("norm", "position", "mixer", "feed_forward", "block", "embedding", "head", "injection")
 _REGISTRIES: Dict[str, Dict[str, type]] = {k: {} for k in _KINDS}
 
 

@@ -61,9 +61,17 @@ class LayerSpec:
 class ScheduleEntry:
     """One run of a layer.  `layer` indexes `ModelSpec.layers` (a layer may be named by several
     entries: same weights, run again).  Each entry keeps memory of its own (cache rows, state)
-    unless `memory_of` names an earlier entry, whose cache it then reads without writing."""
+    unless `memory_of` names an earlier entry, whose cache it then reads without writing.  `inject`: the model's
+    injection part runs right before this entry (a pass over looped layers starts here)."""
     layer: int
     memory_of: Optional[int] = None
+    inject: bool = False
+
+
+def looped_schedule(n_layers: int, start: int, stop: int, times: int, inject: bool = False) -> Tuple[ScheduleEntry, ...]:
+    """Layers 0 .. n_layers - 1 in order, of which start .. stop - 1 run `times` times in a row before the rest follow."""
+    body = [ScheduleEntry(i, inject=inject and i == start) for i in range(start, stop)]
+    return tuple([ScheduleEntry(i) for i in range(start)] + body * times + [ScheduleEntry(i) for i in range(stop, n_layers)])
 
 
 @dataclass(frozen=True)
@@ -87,7 +95,12 @@ class ModelSpec:
     streams: int = 0                            # > 0: the layers work on so many copies of the residual stream, side by side per
                                                 # token ([tokens, streams * width]); they start equal and are summed before the final norm
 
+    injection: Optional[PartSpec] = None        # what the stream passes through before the entries that say `inject`
+    injection_prefix: str = ""
+
     def validate(self) -> None:
+        if self.injection is None and any(e.inject for e in self.schedule):
+            raise ValueError("the schedule injects, but the model has no injection part")
         for i, e in enumerate(self.schedule):
             if not (0 <= e.layer < len(self.layers)):
                 raise ValueError(f"schedule entry {i} names layer {e.layer}, but there are {len(self.layers)} layers")
