@@ -229,6 +229,45 @@ TORUTAR_SIZES = {
 }
 
 
+def _vavupel(width, lat_heads, lat_dim, lat_rot, lat_vdim, kv_rank, window, ret_heads, ret_dim, ret_vdim, ff, buckets, vocab, **_):
+    mlp = {"kind": "dense", "ff": ff}
+    latent = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": lat_heads, "dim": lat_dim, "rot_dim": lat_rot, "vdim": lat_vdim, "kv_rank": kv_rank, "scale": (lat_dim + lat_rot) ** -0.5,
+        "mask": {"size": window}, "rot": {"base": 10000.0, "dims": lat_rot}}}
+    retention = {"type": "retention", "mlp": mlp, "mixer": {
+        "heads": ret_heads, "dim": ret_dim, "vdim": ret_vdim, "rot": {"base": 10000.0, "dims": ret_dim},
+        "decay": [1.0 - 2.0 ** -(1 + 7 * h / max(1, ret_heads - 1)) for h in range(ret_heads)]}}
+    return {"architecture": "Vavupel", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "embedding": {"scale": 1.0, "bigram": {"buckets": buckets, "mul_prev": 31, "mul_cur": 7}},
+            "loop": {"start": 1, "stop": 3, "times": 2}, "layers": [retention, latent, retention, latent]}
+
+
+def _navalorn_dense(z, runs):
+    """The decoder with a latent cache at the same sizes (its own query latent, no window), dense feed-forwards only."""
+    c = _navalorn(z["width"], z["lat_heads"], z["lat_dim"], z["lat_rot"], z["lat_vdim"], z["kv_rank"], z["q_rank"], z["ff"], 2, 1, 64, z["vocab"], 1)
+    return dict(c, layers=[c["layers"][0]] * runs)
+
+
+def _nuzinex_linear(z, pairs):
+    """Linear attention with constant decays at the same sizes beside windowed attention, dense feed-forwards."""
+    c = _nuzinex(z["width"], z["heads"], z["kv"], z["dim"], z["dim"], z["window"], z["ff"], 1, 1, 8, 1, 1, 8, 8, 1, z["ret_heads"], z["ret_dim"],
+                 z["ret_vdim"], 128, z["vocab"])
+    return dict(c, layers=[c["layers"][2], c["layers"][0]] * pairs)
+
+
+# layer sizes of the kind real models have: retention and latent attention in a window in turn, each with a dense feed-forward,
+# the middle two layers run twice (six layer runs).  Beside it, with six layers each: the decoder with a latent cache, the one
+# with linear attention (and windowed attention in turn), and the Llama decoder
+VAVUPEL_SIZES = {
+    "w2048": dict(width=2048, lat_heads=16, lat_dim=128, lat_rot=64, lat_vdim=128, kv_rank=512, q_rank=1536, window=1024, ret_heads=16,
+                  ret_dim=128, ret_vdim=128, ff=8192, buckets=65521, vocab=32000, heads=16, kv=4, dim=128),
+    "w4096": dict(width=4096, lat_heads=32, lat_dim=128, lat_rot=64, lat_vdim=128, kv_rank=512, q_rank=1536, window=2048, ret_heads=32,
+                  ret_dim=128, ret_vdim=128, ff=14336, buckets=65521, vocab=32000, heads=32, kv=8, dim=128),
+    "w2048_odd": dict(width=2048, lat_heads=32, lat_dim=64, lat_rot=32, lat_vdim=40, kv_rank=256, q_rank=768, window=500, ret_heads=12,
+                      ret_dim=96, ret_vdim=64, ff=6144, buckets=40009, vocab=32000, heads=32, kv=8, dim=64),
+}
+
+
 def _barovik_beside(z):
     keys = ("width", "heads", "kv", "dim", "vdim", "chunk", "ff", "ssm_heads", "ssm_dim", "state", "groups", "experts", "top",
             "expert_ff", "shared_ff", "vocab", "pairs")
@@ -236,7 +275,7 @@ def _barovik_beside(z):
 
 
 def measure_hybrid(args):
-    """`--workload barovik` / `--workload navalorn` / `--workload nuzinex` / `--workload torutar`: prompt and decode throughput of that decoder at a few real layer sizes
+    """`--workload barovik` / `--workload navalorn` / `--workload nuzinex` / `--workload torutar` / `--workload vavupel`: prompt and decode throughput of that decoder at a few real layer sizes
     (random weights), beside the Llama decoder with the same width, heads, feed-forward width and number of layers (nuzinex:
     beside the hybrid decoder with windowed attention and state-space layers, and the Llama decoder); and the
     device time per kind of operation for one prompt step and one decode step of each.  One JSON line."""
@@ -323,6 +362,8 @@ def measure_hybrid(args):
         sizes, build, label = NUZINEX_SIZES, _nuzinex, "nuzinex"
     if args.workload == "torutar":
         sizes, build, label = TORUTAR_SIZES, _torutar, "torutar"
+    if args.workload == "vavupel":
+        sizes, build, label = VAVUPEL_SIZES, _vavupel, "vavupel"
     names = [n for n in sizes if not args.sizes or n in args.sizes.split(",")]
     for name in names:
         z = sizes[name]
@@ -330,7 +371,11 @@ def measure_hybrid(args):
         out[name] = {"sizes": z, label: hybrid}
         if label in ("nuzinex", "torutar") and not args.skip_points:
             out[name]["barovik_equal_size"] = one(_barovik_beside(z))
-        if not args.skip_points:
+        if label == "vavupel" and not args.skip_points:
+            out[name]["navalorn_equal_size"] = one(_navalorn_dense(z, 6))
+            out[name]["nuzinex_equal_size"] = one(_nuzinex_linear(z, 3))
+            out[name]["llama_equal_size"] = one(_llama_like(z["width"], z["heads"], z["kv"], z["dim"], z["ff"], z["vocab"], 6))
+        elif not args.skip_points:
             out[name]["llama_equal_size"] = one(_llama_like(z["width"], z["heads"], z["kv"], z["llama_dim"] if latent else z["dim"], z["ff"],
                                                             z["vocab"], 2 * z["pairs"]))
     clocks.stop()
@@ -474,10 +519,10 @@ def main():
     ap.add_argument("--impl", default="ours")
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the named configuration (recorded in config)")
     ap.add_argument("--skip-points", action="store_true")
-    ap.add_argument("--workload", default="8b", choices=["8b", "1b", "3b", "barovik", "navalorn", "nuzinex", "torutar"],
-                    help="8b: the headline; 1b, 3b: the baseline's other workloads; barovik, navalorn, nuzinex, torutar: one of the "
+    ap.add_argument("--workload", default="8b", choices=["8b", "1b", "3b", "barovik", "navalorn", "nuzinex", "torutar", "vavupel"],
+                    help="8b: the headline; 1b, 3b: the baseline's other workloads; barovik, navalorn, nuzinex, torutar, vavupel: one of the "
                          "other decoders beside the Llama decoder at equal layer sizes (--sizes, --batch, --held)")
-    ap.add_argument("--sizes", default="", help="for --workload barovik / navalorn / nuzinex / torutar: which of its sizes to run, with commas (default: all)")
+    ap.add_argument("--sizes", default="", help="for --workload barovik / navalorn / nuzinex / torutar / vavupel: which of its sizes to run, with commas (default: all)")
     ap.add_argument("--tune", default="", help="overrides of kernel choices, e.g. small_skinny=0,attn_waves=2")
     ap.add_argument("--only", default="", choices=["", "prefill", "decode", "timeline"],
                     help="run one phase alone and print its time (a short program for a launch list under a profiler; no bench "
@@ -500,7 +545,7 @@ def main():
         for kv in filter(None, args.tune.split(",")):
             k, v = kv.split("=")
             _ops.TUNE[k] = type(_ops.TUNE[k])(float(v))
-    if args.workload in ("barovik", "navalorn", "nuzinex", "torutar"):
+    if args.workload in ("barovik", "navalorn", "nuzinex", "torutar", "vavupel"):
         return measure_hybrid(args)
     if args.workload != "8b":
         return run_workload(args.workload, args)

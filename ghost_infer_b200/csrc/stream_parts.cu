@@ -222,17 +222,17 @@ norm_gate_kernel(T* __restrict__ out, const float* y, const T* g, long ldg, cons
 
 // The same for groups of up to 512 numbers whose parts start on 16-byte boundaries: a warp takes a group, its lanes four
 // neighbouring numbers at a time, kept in registers between the sum and the result.
-constexpr int NG_VEC = 4;
-template <typename T, typename TW>
+template <typename T, typename TW, int NG_VEC>
 __global__ void __launch_bounds__(256)
 norm_gate_warp_kernel(T* __restrict__ out, const float* y, const T* g, long ldg, const TW* __restrict__ w, int inner, int gs,
-                      int w_per_row, int act, float eps, long total_groups) {
+                      int w_per_row, int act, float eps, unsigned total_groups) {
   gi::pdl_prologue();
-  const long grp = (long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const unsigned grp = blockIdx.x * 8 + (threadIdx.x >> 5);
   if (grp >= total_groups) return;
-  const int lane = threadIdx.x & 31, groups = inner / gs;
-  const size_t t = grp / groups;
-  const int c0 = (int)(grp - (long)t * groups) * gs;
+  const int lane = threadIdx.x & 31;
+  const unsigned groups = inner / gs, tt = grp / groups;
+  const size_t t = tt;
+  const int c0 = (int)(grp - tt * groups) * gs;
   const float* yr = y + t * inner + c0;
   float4 v[NG_VEC], z[NG_VEC];
   float ss = 0.f;
@@ -362,11 +362,14 @@ extern "C" int gi_norm_gate(void* out, int dtype, const float* y, const void* g,
   if (inner <= 0 || group <= 0 || inner % group) return gi::fail(GI_ERR_ARG, "norm_gate: %d values do not divide into groups of %d", inner, group);
   cudaError_t e = cudaSuccess;
   const long total_groups = (long)n_rows * (inner / group);
-  if (group % 4 == 0 && group <= NG_VEC * 128 && ldg % 4 == 0 && (total_groups + 7) / 8 <= 0x7fffffffL &&
+  if (group % 4 == 0 && group <= 512 && ldg % 4 == 0 && total_groups <= 0x7fffff00L &&
       (((uintptr_t)out | (uintptr_t)y | (uintptr_t)g | (uintptr_t)w) & 15) == 0) {
-    GI_DISPATCH_DTYPE(dtype, T, GI_DISPATCH_DTYPE(w_dtype, TW,
-        e = gi::launch(norm_gate_warp_kernel<T, TW>, dim3((unsigned)((total_groups + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, (T*)out, y,
-                       (const T*)g, ldg, (const TW*)w, inner, group, w_per_row, act, eps, total_groups)));
+    const dim3 grid((unsigned)((total_groups + 7) / 8));
+    GI_DISPATCH_DTYPE(dtype, T, GI_DISPATCH_DTYPE(w_dtype, TW, {
+      auto kern = group <= 128 ? norm_gate_warp_kernel<T, TW, 1> : (group <= 256 ? norm_gate_warp_kernel<T, TW, 2> : norm_gate_warp_kernel<T, TW, 4>);
+      e = gi::launch(kern, grid, dim3(256), 0, (cudaStream_t)stream, (T*)out, y, (const T*)g, ldg, (const TW*)w, inner, group, w_per_row,
+                     act, eps, (unsigned)total_groups);
+    }));
     return gi::check(e, "norm_gate");
   }
   GI_DISPATCH_DTYPE(dtype, T, GI_DISPATCH_DTYPE(w_dtype, TW,

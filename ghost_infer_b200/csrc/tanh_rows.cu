@@ -64,12 +64,12 @@ __device__ __forceinline__ float4 tr_add(float4 a, float4 b) { return make_float
 
 template <typename TW, typename TH>
 __global__ void __launch_bounds__(256)
-tanh_rows_kernel(const TanhRows a, long total) {
+tanh_rows_kernel(const TanhRows a, unsigned total) {
   gi::pdl_launch_dependents();
-  const long g = (long)blockIdx.x * blockDim.x + threadIdx.x;
-  const int per = (a.d + 3) / 4;
+  const unsigned g = blockIdx.x * blockDim.x + threadIdx.x;
+  const unsigned per = (a.d + 3) / 4;
   const bool live = g < total;
-  const long r = live ? g / per : 0;
+  const unsigned r = live ? g / per : 0;
   const int c = live ? (int)(g - r * per) * 4 : 0;
   const int n = min(4, a.d - c);
   const float4 z4 = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -79,7 +79,7 @@ tanh_rows_kernel(const TanhRows a, long total) {
   if (a.w2 != nullptr) { w2 = tr_get((const TW*)a.w2 + c, n, a.vec); b2 = tr_get((const TW*)a.b2 + c, n, a.vec); }
   gi_settle_span sp = {0, 0, 0};
   if (a.settle_of) sp = gi_span_of(a.st, c);
-  const long m = a.rows != nullptr ? gi::ld_step(a.rows + r) : r;
+  const long m = a.rows != nullptr ? gi::ld_step(a.rows + r) : (long)r;
   gi::pdl_wait();
   if (!live) return;
   float4 v = z4;
@@ -102,7 +102,7 @@ tanh_rows_kernel(const TanhRows a, long total) {
   }
   if (a.h != nullptr) {
     if (a.w2 != nullptr) v = tr_norm(v, a.a2, w2, b2);
-    tr_put((TH*)a.h + r * a.d + c, v, n, a.vec);
+    tr_put((TH*)a.h + (size_t)r * a.d + c, v, n, a.vec);
   }
 }
 
@@ -171,10 +171,10 @@ extern "C" int gi_tanh_rows(const float* x, long ldx, const int* rows, float* y,
   const long total = (long)n_rows * ((d + 3) / 4);
   const int threads = total <= 148L * 256 ? 64 : 256;      // few rows: more blocks, so that every SM takes part
   const long blocks = (total + threads - 1) / threads;
-  if (blocks > 0x7fffffffL) return gi::fail(GI_ERR_UNSUPPORTED, "tanh rows: too many rows for one launch");
+  if (total > 0x7fffff00L) return gi::fail(GI_ERR_UNSUPPORTED, "tanh rows: too many rows for one launch");
   cudaError_t e = cudaSuccess;
   GI_DISPATCH_DTYPE(w_dtype, TW, GI_DISPATCH_DTYPE(h_dtype, TH,
-      e = gi::launch(tanh_rows_kernel<TW, TH>, dim3((unsigned)blocks), dim3(threads), 0, (cudaStream_t)stream, a, total)));
+      e = gi::launch(tanh_rows_kernel<TW, TH>, dim3((unsigned)blocks), dim3(threads), 0, (cudaStream_t)stream, a, (unsigned)total)));
   return gi::check(e, "tanh rows");
 }
 

@@ -3,12 +3,25 @@
 It shares no code with the library: the tests compare the library's logits and intermediate results with what these
 functions give for the same configuration dict and the same tensors (name -> array).  Notation: T tokens, d the width,
 H heads; matrices are stored [out, in] and applied as x @ W.T.
+
+`act` (everywhere optional) is applied to whatever a 16-bit run keeps in 16 bits between its steps: the identity here; a test
+that passes small random changes learns how far roundings may move each position's logits (`shaken`).
 """
 from __future__ import annotations
 
 import math
 
 import numpy as np
+
+
+def exactly(a):
+    return a
+
+
+def shaken(seed, size=2.0 ** -8):
+    """An `act` that changes every number by up to half of `size` of itself, as rounding to 8 significant bits does."""
+    rng = np.random.default_rng(seed)
+    return lambda a: a * (1.0 + size * (rng.random(np.shape(a)) - 0.5))
 
 
 def rms_unit(x, eps):
@@ -73,13 +86,13 @@ def softmax_with_sink(s, sink):
     return p / (p.sum(axis=1, keepdims=True) + np.exp(sink - top))
 
 
-def latent_attention(h, positions, W, pre, m, eps):
+def latent_attention(h, positions, W, pre, m, eps, act=exactly):
     T, H, n, r, mv, rank = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
-    q = (h @ W[pre + "q"].T).reshape(T, H, n + r)
-    down = h @ W[pre + "dkv"].T
-    c = rms_unit(down[:, :rank], eps) * W[pre + "dkv.norm"]
-    k_rot = rotate(down[:, rank:], positions, m["rot"]["dims"], m["rot"]["base"], "adjacent")        # [T, r], all heads share it
-    q_rot = rotate(q[:, :, n:], positions, m["rot"]["dims"], m["rot"]["base"], "adjacent")
+    q = act(h @ W[pre + "q"].T).reshape(T, H, n + r)
+    down = act(h @ W[pre + "dkv"].T)
+    c = act(rms_unit(down[:, :rank], eps) * W[pre + "dkv.norm"])
+    k_rot = act(rotate(down[:, rank:], positions, m["rot"]["dims"], m["rot"]["base"], "adjacent"))   # [T, r], all heads share it
+    q_rot = act(rotate(q[:, :, n:], positions, m["rot"]["dims"], m["rot"]["base"], "adjacent"))
     k = (c @ W[pre + "uk"].T).reshape(T, H, n)
     v = (c @ W[pre + "uv"].T).reshape(T, H, mv)
     mask = visible(T, m["mask"]["size"] if m.get("mask") else None)
@@ -87,34 +100,34 @@ def latent_attention(h, positions, W, pre, m, eps):
     for a in range(H):
         s = (q[:, a, :n] @ k[:, a].T + q_rot[:, a] @ k_rot.T) * m["scale"]
         out[:, a] = softmax_with_sink(np.where(mask, s, -np.inf), float(W[pre + "sink"][a])) @ v[:, a]
-    out = out * sigmoid(h @ W[pre + "g"].T)[:, :, None]
+    out = act(act(out) * sigmoid(act(h @ W[pre + "g"].T))[:, :, None])
     return out.reshape(T, H * mv) @ W[pre + "o"].T
 
 
-def retention(h, positions, W, pre, m, eps, state=None):
+def retention(h, positions, W, pre, m, eps, state=None, act=exactly):
     """Linear attention with a constant decay per head.  `state` [H, n, mv] is carried in and returned."""
     T, H, n, mv = h.shape[0], m["heads"], m["dim"], m["vdim"]
-    q = rotate((h @ W[pre + "q"].T).reshape(T, H, n), positions, m["rot"]["dims"], m["rot"]["base"], "half")
-    k = rotate((h @ W[pre + "k"].T).reshape(T, H, n), positions, m["rot"]["dims"], m["rot"]["base"], "half") * n ** -0.5
-    v = (h @ W[pre + "v"].T).reshape(T, H, mv)
+    q = rotate(act(h @ W[pre + "q"].T).reshape(T, H, n), positions, m["rot"]["dims"], m["rot"]["base"], "half")
+    k = rotate(act(h @ W[pre + "k"].T).reshape(T, H, n), positions, m["rot"]["dims"], m["rot"]["base"], "half") * n ** -0.5
+    v = act(h @ W[pre + "v"].T).reshape(T, H, mv)
     S = np.zeros((H, n, mv)) if state is None else state.copy()
     decay = np.asarray(m["decay"], dtype=np.float64)[:, None, None]
     o = np.zeros((T, H, mv))
     for t in range(T):
         S = decay * S + k[t][:, :, None] * v[t][:, None, :]
         o[t] = np.einsum("hnm,hn->hm", S, q[t])
-    g = h @ W[pre + "g"].T
-    o = rms_unit(o, eps).reshape(T, H * mv) * (g * sigmoid(g))
+    g = act(h @ W[pre + "g"].T)
+    o = act(rms_unit(o, eps).reshape(T, H * mv) * (g * sigmoid(g)))
     return o @ W[pre + "o"].T, S
 
 
-def squared_relu_mlp(h, W, pre):
-    return np.maximum(h @ W[pre + "up"].T, 0.0) ** 2 @ W[pre + "down"].T
+def squared_relu_mlp(h, W, pre, act=exactly):
+    return act(np.maximum(h @ W[pre + "up"].T, 0.0) ** 2) @ W[pre + "down"].T
 
 
-def injected(x, x0, W):
+def injected(x, x0, W, act=exactly):
     """What a pass over the looped layers starts from: a product of the stream beside the embedding output."""
-    return np.concatenate([x, x0], axis=1) @ W["loop.in"].T
+    return act(np.concatenate([x, x0], axis=1)) @ W["loop.in"].T
 
 
 def softcap(z, cap):
@@ -130,20 +143,20 @@ def runs(cfg):
     return [(i, False) for i in range(loop["start"])] + body * loop["times"] + [(i, False) for i in range(loop["stop"], n)]
 
 
-def layer(x, i, cfg, W, positions):
+def layer(x, i, cfg, W, positions, act=exactly):
     lp, lay, eps = f"l{i}.", cfg["layers"][i], cfg["norm"]["eps"]
-    h = tanh_norm(x, W, lp + "norm1")
+    h = act(tanh_norm(x, W, lp + "norm1"))
     if lay["type"] == "retention":
-        y = retention(h, positions, W, lp + "mix.", lay["mixer"], eps)[0]
+        y = retention(h, positions, W, lp + "mix.", lay["mixer"], eps, act=act)[0]
     else:
-        y = latent_attention(h, positions, W, lp + "mix.", lay["mixer"], eps)
+        y = latent_attention(h, positions, W, lp + "mix.", lay["mixer"], eps, act)
     x = x + tanh_norm(y, W, lp + "norm1b")
     if lay.get("mlp") is not None:
-        x = x + tanh_norm(squared_relu_mlp(tanh_norm(x, W, lp + "norm2"), W, lp + "mlp."), W, lp + "norm2b")
+        x = x + tanh_norm(squared_relu_mlp(act(tanh_norm(x, W, lp + "norm2")), W, lp + "mlp.", act), W, lp + "norm2b")
     return x
 
 
-def forward(cfg, W, tokens, return_layers=False):
+def forward(cfg, W, tokens, return_layers=False, act=exactly):
     """Logits [T, vocab] of one sequence from its first token (float64); optionally the stream after every layer run."""
     W = {k: np.asarray(v, dtype=np.float64) for k, v in W.items()}
     positions = np.arange(len(tokens))
@@ -151,10 +164,10 @@ def forward(cfg, W, tokens, return_layers=False):
     x, after = x0, []
     for i, starts_pass in runs(cfg):
         if starts_pass:
-            x = injected(x, x0, W)
-        x = layer(x, i, cfg, W, positions)
+            x = injected(x, x0, W, act)
+        x = layer(x, i, cfg, W, positions, act)
         after.append(x)
-    logits = softcap(tanh_norm(x, W, "final.norm") @ W["head"].T, cfg.get("logit_softcap"))
+    logits = softcap(act(tanh_norm(x, W, "final.norm")) @ W["head"].T, cfg.get("logit_softcap"))
     return (logits, np.stack(after)) if return_layers else logits
 
 
