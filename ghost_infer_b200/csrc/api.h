@@ -573,11 +573,11 @@ int gi_attn_decode_generic_ex3(void* out, long ldo, float* part_o, float* part_m
 // v = x + n1(y) per row of d float32 numbers (x or y may be null; rows ldx / ldy apart); n1(u) = tanh(alpha1 u) * w1 + b1, or u
 // (w1 null).  x_out (or null; rows side by side, may be x): v, or `base` (rows ldb apart) in its place.  zero_y: y is zero
 // afterwards.  h (or null; rows side by side, in h_dtype): n2(v) likewise.  `rows` (with neither y nor x_out): the rows of x to
-// read.  settle_of 1 / 2: `settle` describes partial sums pending for x / y (rows of one deferred product's output; they are
+// read.  quick: tanh by the approximate instructions (a few units in the last place).  settle_of 1 / 2: `settle` describes partial sums pending for x / y (rows of one deferred product's output; they are
 // added to what is read).
 int gi_tanh_rows(const float* x, long ldx, const int* rows, float* y, long ldy, int zero_y, float* x_out, const float* base,
                  long ldb, float alpha1, const void* w1, const void* b1, float alpha2, const void* w2, const void* b2, int w_dtype,
-                 void* h, int h_dtype, int n_rows, int d, int settle_of, gi_settle_t settle, void* stream);
+                 void* h, int h_dtype, int n_rows, int d, int quick, int settle_of, gi_settle_t settle, void* stream);
 // x = cap * tanh(x / cap), float32, in place.
 int gi_softcap_rows(float* x, float cap, long n_values, void* stream);
 // out[t] = table[token_t] * scale + pairs[(prev_t * mul_prev + token_t * mul_cur) mod buckets] (row `buckets` at position 0).

@@ -56,13 +56,26 @@ __device__ __forceinline__ void tr_put(T* p, float4 v, int n, int vec) {
   if (n > 2) gi::stf(p + 2, v.z);
   if (n > 3) gi::stf(p + 3, v.w);
 }
+// The tanh of the 16-bit path: gi::tanh_fast (good to about 1e-7 of 1), and below 0.2, where that would lose relative accuracy,
+// the first four terms of the series x - x^3/3 + 2 x^5/15 - 17 x^7/315: a few units in the last place of a float everywhere, at a
+// third of tanhf's instructions and without its branch, which leaves the pass to the memory.
+template <bool QUICK>
+__device__ __forceinline__ float tr_tanh(float x) {
+  if (!QUICK) return tanhf(x);
+  const float q = x * x;
+  const float series = x * fmaf(q, fmaf(q, fmaf(q, -17.0f / 315.0f, 2.0f / 15.0f), -1.0f / 3.0f), 1.0f);
+  const float wide = gi::tanh_fast(fminf(fmaxf(x, -16.0f), 16.0f));      // beyond, tanh is 1 to the last bit
+  return fabsf(x) < 0.2f ? series : wide;
+}
+template <bool QUICK>
 __device__ __forceinline__ float4 tr_norm(float4 v, float alpha, float4 w, float4 b) {
-  return make_float4(fmaf(tanhf(alpha * v.x), w.x, b.x), fmaf(tanhf(alpha * v.y), w.y, b.y), fmaf(tanhf(alpha * v.z), w.z, b.z),
-                     fmaf(tanhf(alpha * v.w), w.w, b.w));
+  return make_float4(fmaf(tr_tanh<QUICK>(alpha * v.x), w.x, b.x), fmaf(tr_tanh<QUICK>(alpha * v.y), w.y, b.y),
+                     fmaf(tr_tanh<QUICK>(alpha * v.z), w.z, b.z), fmaf(tr_tanh<QUICK>(alpha * v.w), w.w, b.w));
 }
 __device__ __forceinline__ float4 tr_add(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
 
-template <typename TW, typename TH>
+// SETTLE: some row has sums pending (their loads in flight cost registers the plain pass does without).
+template <typename TW, typename TH, bool QUICK, bool SETTLE>
 __global__ void __launch_bounds__(256)
 tanh_rows_kernel(const TanhRows a, unsigned total) {
   gi::pdl_launch_dependents();
@@ -78,20 +91,20 @@ tanh_rows_kernel(const TanhRows a, unsigned total) {
   if (a.w1 != nullptr) { w1 = tr_get((const TW*)a.w1 + c, n, a.vec); b1 = tr_get((const TW*)a.b1 + c, n, a.vec); }
   if (a.w2 != nullptr) { w2 = tr_get((const TW*)a.w2 + c, n, a.vec); b2 = tr_get((const TW*)a.b2 + c, n, a.vec); }
   gi_settle_span sp = {0, 0, 0};
-  if (a.settle_of) sp = gi_span_of(a.st, c);
+  if (SETTLE) sp = gi_span_of(a.st, c);
   const long m = a.rows != nullptr ? gi::ld_step(a.rows + r) : (long)r;
   gi::pdl_wait();
   if (!live) return;
-  float4 v = z4;
+  float* yp = a.y + m * a.ldy + c;
+  float4 v = z4, u = z4;
+  if (a.x != nullptr) v = tr_get(a.x + m * a.ldx + c, n, a.vec);
+  if (a.y != nullptr) u = tr_get((const float*)yp, n, a.vec);
   if (a.x != nullptr) {
-    v = tr_get(a.x + m * a.ldx + c, n, a.vec);
-    if (a.settle_of == 1 && sp.c_first != sp.c_last) v = tr_add(v, gi_sum_pieces4(a.st, sp, (int)m, c));
+    if (SETTLE && a.settle_of == 1 && sp.c_first != sp.c_last) v = tr_add(v, gi_sum_pieces4(a.st, sp, (int)m, c));
   }
   if (a.y != nullptr) {
-    float* yp = a.y + m * a.ldy + c;
-    float4 u = tr_get((const float*)yp, n, a.vec);
-    if (a.settle_of == 2 && sp.c_first != sp.c_last) u = tr_add(u, gi_sum_pieces4(a.st, sp, (int)m, c));
-    if (a.w1 != nullptr) u = tr_norm(u, a.a1, w1, b1);
+    if (SETTLE && a.settle_of == 2 && sp.c_first != sp.c_last) u = tr_add(u, gi_sum_pieces4(a.st, sp, (int)m, c));
+    if (a.w1 != nullptr) u = tr_norm<QUICK>(u, a.a1, w1, b1);
     v = a.x != nullptr ? tr_add(v, u) : u;
     if (a.zero_y) tr_put(yp, z4, n, a.vec);
   }
@@ -101,7 +114,7 @@ tanh_rows_kernel(const TanhRows a, unsigned total) {
     tr_put(a.x_out + m * a.d + c, o, n, a.vec);
   }
   if (a.h != nullptr) {
-    if (a.w2 != nullptr) v = tr_norm(v, a.a2, w2, b2);
+    if (a.w2 != nullptr) v = tr_norm<QUICK>(v, a.a2, w2, b2);
     tr_put((TH*)a.h + (size_t)r * a.d + c, v, n, a.vec);
   }
 }
@@ -153,7 +166,7 @@ embed_pair_kernel(float* __restrict__ out, const TW* __restrict__ table, const T
 
 extern "C" int gi_tanh_rows(const float* x, long ldx, const int* rows, float* y, long ldy, int zero_y, float* x_out, const float* base,
                             long ldb, float alpha1, const void* w1, const void* b1, float alpha2, const void* w2, const void* b2,
-                            int w_dtype, void* h, int h_dtype, int n_rows, int d, int settle_of, gi_settle_t settle, void* stream) {
+                            int w_dtype, void* h, int h_dtype, int n_rows, int d, int quick, int settle_of, gi_settle_t settle, void* stream) {
   if (n_rows <= 0) return GI_OK;
   if (d <= 0 || (!x && !y)) return gi::fail(GI_ERR_ARG, "tanh rows: bad width %d or nothing to read", d);
   if ((w1 && !b1) || (w2 && !b2)) return gi::fail(GI_ERR_ARG, "tanh rows: a norm needs its weight and its bias");
@@ -173,8 +186,11 @@ extern "C" int gi_tanh_rows(const float* x, long ldx, const int* rows, float* y,
   const long blocks = (total + threads - 1) / threads;
   if (total > 0x7fffff00L) return gi::fail(GI_ERR_UNSUPPORTED, "tanh rows: too many rows for one launch");
   cudaError_t e = cudaSuccess;
-  GI_DISPATCH_DTYPE(w_dtype, TW, GI_DISPATCH_DTYPE(h_dtype, TH,
-      e = gi::launch(tanh_rows_kernel<TW, TH>, dim3((unsigned)blocks), dim3(threads), 0, (cudaStream_t)stream, a, (unsigned)total)));
+  GI_DISPATCH_DTYPE(w_dtype, TW, GI_DISPATCH_DTYPE(h_dtype, TH, {
+    auto kern = a.settle_of ? (quick ? tanh_rows_kernel<TW, TH, true, true> : tanh_rows_kernel<TW, TH, false, true>)
+                            : (quick ? tanh_rows_kernel<TW, TH, true, false> : tanh_rows_kernel<TW, TH, false, false>);
+    e = gi::launch(kern, dim3((unsigned)blocks), dim3(threads), 0, (cudaStream_t)stream, a, (unsigned)total);
+  }));
   return gi::check(e, "tanh rows");
 }
 

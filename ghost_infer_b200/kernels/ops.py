@@ -136,7 +136,7 @@ def _bind():
         "gi_moe_route_shares": [P, P, P, P, I, L, P, P, I, I, I, I, I, I, P, F, P],
         "gi_moe_gemm_gate_up_clamped": [P, I, P, L, P, I, L, P, P, I, I, I, I, I, I, F, F, P],
         "gi_attn_prefill_generic_ex3": [P, L, P, L, I, P, P, P, I, P, P, P, I, I, I, I, I, F, I, I, F, P, I, L, I, P],
-        "gi_tanh_rows": [P, L, P, P, L, I, P, P, L, F, P, P, F, P, P, I, P, I, I, I, I, SettleT, P],
+        "gi_tanh_rows": [P, L, P, P, L, I, P, P, L, F, P, P, F, P, P, I, P, I, I, I, I, I, SettleT, P],
         "gi_softcap_rows": [P, F, L, P],
         "gi_embed_pair": [P, P, P, I, P, P, P, P, I, P, L, I, I, I, F, I, LL, LL, P],
         "gi_latent_prepare_q": [P, P, I, L, P, P, I, F, P, I, P, P, P, I, P, I, I, I, I, I, P, L, P, L, I, I, P],
@@ -2450,11 +2450,12 @@ def moe_route_shares(h: torch.Tensor, w_router: torch.Tensor, top: int, correcti
 # ---- streams with element-wise tanh norms, embeddings of token pairs, rotated linear attention ---------------------------
 def tanh_rows(x: Optional[torch.Tensor], y: Optional[torch.Tensor], post, pre, out_dtype: Optional[torch.dtype], *,
               x_out: Optional[torch.Tensor] = None, base: Optional[torch.Tensor] = None, zero_y: bool = False,
-              rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+              rows: Optional[torch.Tensor] = None, quick: bool = False) -> Optional[torch.Tensor]:
     """v = x + post(y); `x_out` receives v (or `base` in its place); returns pre(v) in `out_dtype` (None: nothing).  x, y:
     float32 rows, either may be None; `post` and `pre`: (alpha, weight, bias) of a norm tanh(alpha u) * weight + bias, or None
     for the value itself.  `zero_y`: y is zero afterwards.  `rows` (with x alone): the rows to read.  Partial sums that a
-    deferred product left for x or for y are added on the way (and stay in x only where `x_out` writes it back)."""
+    deferred product left for x or for y are added on the way (and stay in x only where `x_out` writes it back).  `quick`: the
+    16-bit path's tanh (a few units in the last place of a float instead of one)."""
     lib = _bind()
     src = x if x is not None else y
     if src is None:
@@ -2494,7 +2495,7 @@ def tanh_rows(x: Optional[torch.Tensor], y: Optional[torch.Tensor], post, pre, o
     ld = lambda t: t.stride(0) if t is not None else d
     _check(lib, lib.gi_tanh_rows(ptr(x), ld(x), _i32(rows, "rows"), ptr(y), ld(y), int(zero_y), ptr(x_out), ptr(base), ld(base),
                                  float(a1), ptr(w1), ptr(b1), float(a2), ptr(w2), ptr(b2), _DT[wdt] if wdt is not None else F32,
-                                 ptr(h), _dt(h, "normed rows") if h is not None else F32, n, d, settle_of, rec, _stream()))
+                                 ptr(h), _dt(h, "normed rows") if h is not None else F32, n, d, int(quick), settle_of, rec, _stream()))
     return h
 
 

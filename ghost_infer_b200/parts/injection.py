@@ -61,7 +61,8 @@ class InputInjection(Injection):
             reader = step.next_reader
             read = reader.stream_read(step) if reader is not None else None
             with ops.bucket("norm"):
-                h = ops.tanh_rows(first, base, None, read.norm if read else None, read.dtype if read else None, x_out=x)
+                h = ops.tanh_rows(first, base, None, read.norm if read else None, read.dtype if read else None, x_out=x,
+                                  quick=self.rt.dtype != torch.float32)
             if h is not None:
                 ops.hand_on(x, reader, h)
             return

@@ -135,7 +135,7 @@ class DynamicTanh(Norm):
         with ops.bucket("norm"):
             # sums pending for the stream stay in it, unless only chosen rows are read (whoever does that is its last reader)
             keep = x if rows is None and ops.has_pending(x) else None
-            return ops.tanh_rows(x, None, None, self.numbers, want, rows=rows, x_out=keep)
+            return ops.tanh_rows(x, None, None, self.numbers, want, rows=rows, x_out=keep, quick=self.rt.dtype != torch.float32)
 
     def start_stream(self, e: torch.Tensor, step) -> torch.Tensor:
         x = ops.as_carrier(e)
@@ -149,6 +149,6 @@ class DynamicTanh(Norm):
         read = reader.stream_read(step) if reader is not None else None
         with ops.bucket("norm"):
             h = ops.tanh_rows(x, y, self.numbers, read.norm if read is not None else None, read.dtype if read is not None else None,
-                              x_out=out, base=read.base if read is not None else None, zero_y=zero_y)
+                              x_out=out, base=read.base if read is not None else None, zero_y=zero_y, quick=self.rt.dtype != torch.float32)
         if h is not None:
             ops.hand_on(out, reader, h)

@@ -196,6 +196,11 @@ def test_the_pass_that_joins_and_reads_the_stream(rows, width):
     assert float(y1.abs().max()) == 0.0
     h16 = ops.tanh_rows(x.clone(), y.clone(), post, pre, torch.bfloat16, x_out=x1)
     assert torch.equal(h16, h.bfloat16())
+    # the 16-bit path's tanh, over small and large numbers: a few units in the last place, relative
+    span = x * torch.logspace(-6, 1.5, rows, device="cuda:0")[:, None]
+    unit = (1.0, torch.ones((width,), device="cuda:0"), torch.zeros((width,), device="cuda:0"))
+    torch.testing.assert_close(ops.tanh_rows(span, None, None, unit, torch.float32, quick=True).double(), torch.tanh(span.double()), rtol=1.5e-6, atol=0.0)
+    close(ops.tanh_rows(x.clone(), y.clone(), post, pre, torch.float32, quick=True), plain_norm(want, pre))
     # rows ready made in the stream's place, the sum handed on as it is
     base, x2 = wide[:, width:], x.clone()
     h = ops.tanh_rows(x2, y, post, None, torch.float32, x_out=x2, base=base)
