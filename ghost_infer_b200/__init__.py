@@ -24,11 +24,14 @@ register_architecture("Torutar", TorutarConfig.from_dict, build_torutar_spec, re
 from .config.vavupel import VavupelConfig, build_vavupel_spec
 
 register_architecture("Vavupel", VavupelConfig.from_dict, build_vavupel_spec, replace=True)
+from .config.sofopel import SofopelConfig, build_sofopel_spec
+
+register_architecture("Sofopel", SofopelConfig.from_dict, build_sofopel_spec, replace=True)
 
 from .engine import Engine, Model, StepEntry  # noqa: E402
 from .api import LLM  # noqa: E402
 from .sampling import SamplingParams  # noqa: E402
 
-__all__ = ["ConfigError", "LlamaConfig", "BarovikConfig", "NavalornConfig", "NuzinexConfig", "TorutarConfig", "VavupelConfig", "UnknownArchitectureError", "load_config", "register_architecture",
+__all__ = ["ConfigError", "LlamaConfig", "BarovikConfig", "NavalornConfig", "NuzinexConfig", "TorutarConfig", "VavupelConfig", "SofopelConfig", "UnknownArchitectureError", "load_config", "register_architecture",
            "registered_architectures", "Engine", "Model", "StepEntry", "LLM", "SamplingParams"]
 __version__ = "0.1.0"

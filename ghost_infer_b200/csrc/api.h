@@ -609,6 +609,30 @@ int gi_linear_state_rot(float* o, const void* q, long ldq, const void* k, long l
                         int state_rows, const int* cu_seqlens, const int* seq_slots, int n_seqs, int heads, int K, int V,
                         int n_tokens, void* stream);
 
+// ---- a stream joined once a layer; heads that are the difference of two maps; decays per key channel ------------------------
+// x += scale * y (float32 rows of d numbers side by side; `settle`: partial sums pending for y), y = 0, and, unless h is null,
+// h = x / sqrt(mean(x^2) + eps) * w in h_dtype.
+int gi_join_rows(float* x, float* y, float scale, void* h, int h_dtype, const void* w, int w_dtype, int n_rows, int d, float eps,
+                 gi_settle_t settle, void* stream);
+// Float32 rows [q: heads x 2 x n | k: kv_heads x 2 x n | v: kv_heads x m] through a causal convolution (conv [taps][channels], or
+// taps 0; older inputs in `state`, (taps - 1) * channels floats a slot, oldest first), maps of q and k turned by `table`
+// ([tokens][half] (cos, sin)); q: rows [heads][2][2n], each map's query with zeros in the other's place; keys (both maps side by
+// side) and values to the paged cache.  one_token_each: the state is renewed too (in other steps by gi_mamba2_conv_update).
+int gi_map_prepare(void* q, long ldq, int dtype, const float* in, long ld, const float* conv, int taps, float* state, long state_ld,
+                   int state_rows, int one_token_each, const float* table, int half, int adjacent, const int* positions,
+                   const int* slots, const int* block_table, int max_pages, void* kcache, void* vcache, int n_tokens, int heads,
+                   int kv_heads, int n, int m, void* stream);
+// out[t][h] = factor * v / sqrt(mean(v^2) + eps), v = in[t][h][0] - weight * in[t][h][1] (m numbers each).
+int gi_map_difference(void* out, const void* in, int dtype, int n_rows, int heads, int m, float weight, float factor, float eps,
+                      void* stream);
+// g[t][c] = sigmoid(sum_r low[t][r] up[r][c] + b[c])^(1 / tau).
+int gi_key_decays(float* g, const void* low, long ldl, int dtype, const float* up, const float* b, int n_tokens, int rank,
+                  int channels, float tau, void* stream);
+// gi_linear_state with decays per token and key channel (float32 [tokens][heads * K]) and q times q_scale.
+int gi_linear_state_keyed(float* o, const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, int dtype,
+                          const float* decay, float q_scale, float* state, long state_ld, int state_rows, const int* cu_seqlens,
+                          const int* seq_slots, int n_seqs, int heads, int K, int V, int n_tokens, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

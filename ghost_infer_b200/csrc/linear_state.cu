@@ -1,5 +1,5 @@
 // Linear attention with a matrix of state per head: the entry points of the delta rule, of constant decays and of ready-made
-// gates (linear_state.cuh holds the kernel; linear_state_rot.cu the form whose queries and keys turn).
+// gates (linear_state.cuh holds the kernel; linear_state_rot.cu the form whose queries and keys turn, linear_state_keyed.cu the one with decays per key).
 #include "linear_state.cuh"
 
 extern "C" int gi_linear_state(float* o, const void* q, long ldq, const void* k, long ldk, const void* v, long ldv,

@@ -25,6 +25,8 @@
 // of the block per chunk.
 // ROT: queries and keys turn on the way in: once a chunk's rows are in shared memory the preparing threads turn the pairs of
 // their first numbers by the step's table of angles (loaded with the rows), keys having been scaled when they were stored.
+// KEYED: the decay is a number per token and key channel (ready made, float32 rows [heads * K]), S <- diag(g_t) S + k_t v_t^T,
+// and goes through shared memory beside queries and keys; queries are multiplied by a constant on the way in.
 // State per slot: [heads][V][K] floats (a column's rows side by side) at the start of the slot's row; slot -1 (a padding row
 // of a fixed-size launch) uses the last row of the matrix.
 #pragma once
@@ -88,6 +90,7 @@ struct LsArgs {
   const float2* table;                   // ROT: [tokens][half] (cos, sin)
   int half, adjacent;                    // pairs that turn: (i, i + half), or neighbours
   float k_scale;
+  const float* g_key;                    // KEYED: [tokens][heads * K] decays
 };
 
 // tokens per chunk: two buffers of it stay under 48 KB of shared memory
@@ -96,14 +99,16 @@ template <int KR> struct LsChunk { static constexpr int value = KR >= 32 ? 8 : 1
 // WALK: the step holds sequences of many tokens, and eight whole tokens run without a test between them; without it (steps
 // of one token a sequence) the kernel is the same but smaller, so that two blocks fit an SM at every tile width.
 // Two blocks an SM for the narrower tiles too: a grid of about as many blocks as SMs times two then runs as one round.
-template <typename T, int KR, int COLS, bool DELTA, bool WALK, bool ROT>
+template <typename T, int KR, int COLS, bool DELTA, bool WALK, bool ROT, bool KEYED>
 __global__ void __launch_bounds__(COLS * LS_LANES + LS_PREP, (COLS <= 16 || !WALK) ? 2 : 1)
 linear_state_kernel(const LsArgs a) {
   constexpr int Kp = KR * LS_LANES;            // rows with padding
   constexpr int M = KR / 4;                    // groups of four rows per lane; also a preparing lane's share of a row
   constexpr int NC = COLS * LS_LANES;          // threads that hold S
   constexpr int CH = LsChunk<KR>::value;
-  constexpr int BUF = 2 * CH * Kp + 2 * CH * COLS + 2 * CH;
+  constexpr int BUF = 2 * CH * Kp + 2 * CH * COLS + 2 * CH + (KEYED ? CH * Kp : 0);     // the decays come last
+  constexpr int KEYS_AT = 2 * CH * Kp + 2 * CH * COLS + 2 * CH;
+  static_assert(KEYS_AT % 4 == 0, "the decays start on a 16-byte boundary");
   constexpr int VW = 16 / (int)sizeof(T);      // numbers of a row in sixteen bytes
   static_assert(CH % LS_TB == 0 && CH <= LS_PREP && (CH * Kp) % LS_PREP == 0 && COLS % VW == 0 && CH * COLS / VW <= LS_PREP,
                 "whole exchanges; a preparing thread per token, and per group of a chunk's values");
@@ -150,6 +155,31 @@ linear_state_kernel(const LsArgs a) {
         cs[i] = g < n * a.half ? a.table[(tokc + g / a.half) * a.half + g % a.half] : make_float2(1.f, 0.f);
       }
     }
+    // per-key decays: loaded with the rows, stored with them (sixteen bytes a thread where K allows it)
+    constexpr int DG = KEYED ? (CH * Kp / 4 + LS_PREP - 1) / LS_PREP : 1;
+    float4 dr[DG];
+    if (KEYED) {
+      const int gpr = (K + 3) / 4, total = n * gpr;
+      const size_t ldg = (size_t)a.heads * K;
+#pragma unroll
+      for (int i = 0; i < DG; ++i) {
+        const int g = pt + i * LS_PREP;
+        dr[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (g < total) {
+          const int t = g / gpr, r0 = (g - t * gpr) * 4;
+          const float* p = a.g_key + (tokc + t) * ldg + (size_t)h * K + r0;
+          if (K % 4 == 0) {
+            dr[i] = *reinterpret_cast<const float4*>(p);
+          } else {
+            dr[i].x = p[0];
+            if (r0 + 1 < K) dr[i].y = p[1];
+            if (r0 + 2 < K) dr[i].z = p[2];
+            if (r0 + 3 < K) dr[i].w = p[3];
+          }
+        }
+      }
+    }
+    const float qs = KEYED ? a.q_scale : 1.0f;
     if (a.vec_in) {
       constexpr int QG = (CH * Kp / VW + LS_PREP - 1) / LS_PREP;     // groups of VW numbers a thread moves, per operand
       const int gpr = K / VW, total = n * gpr;
@@ -181,6 +211,7 @@ linear_state_kernel(const LsArgs a) {
               k4.x = ls_silu(k4.x); k4.y = ls_silu(k4.y); k4.z = ls_silu(k4.z); k4.w = ls_silu(k4.w);
             }
             if (ROT) { k4.x *= a.k_scale; k4.y *= a.k_scale; k4.z *= a.k_scale; k4.w *= a.k_scale; }
+            if (KEYED) { q4.x *= qs; q4.y *= qs; q4.z *= qs; q4.w *= qs; }
             *reinterpret_cast<float4*>(sq + t * Kp + r0 + e) = q4;
             *reinterpret_cast<float4*>(sk + t * Kp + r0 + e) = k4;
           }
@@ -213,7 +244,7 @@ linear_state_kernel(const LsArgs a) {
         const int e = pt + i * LS_PREP;
         if (e < total) {
           const int t = e / K, r = e - t * K;
-          sq[t * Kp + r] = act ? ls_silu(qr[i]) : qr[i];
+          sq[t * Kp + r] = (act ? ls_silu(qr[i]) : qr[i]) * qs;
           sk[t * Kp + r] = (act ? ls_silu(kr[i]) : kr[i]) * (ROT ? a.k_scale : 1.0f);
         }
       }
@@ -223,7 +254,19 @@ linear_state_kernel(const LsArgs a) {
         if (e < n * COLS) sv[e] = act ? ls_silu(vr[i]) : vr[i];
       }
     }
-    if (pt < n) {
+    if (KEYED) {
+      float* sd = buf + KEYS_AT;
+      const int gpr = (K + 3) / 4, total = n * gpr;
+#pragma unroll
+      for (int i = 0; i < DG; ++i) {
+        const int g = pt + i * LS_PREP;
+        if (g < total) {
+          const int t = g / gpr;
+          *reinterpret_cast<float4*>(sd + t * Kp + (g - t * gpr) * 4) = dr[i];       // numbers past K: zeros, inside the padding
+        }
+      }
+    }
+    if (pt < n && !KEYED) {
       sg[pt] = ap != nullptr ? expf(-rate * ls_softplus(av + bias)) : dc;
       sb[pt] = bp != nullptr ? 1.0f / (1.0f + expf(-bv)) : 1.0f;
       if (a.g_direct != nullptr) sg[pt] = a.g_direct[(tokc + pt) * a.heads + h];
@@ -287,6 +330,11 @@ linear_state_kernel(const LsArgs a) {
       for (int e = tid - NC; e < 2 * CH * Kp; e += LS_PREP) {
         if (e % Kp >= K) { sm[e] = 0.f; sm[BUF + e] = 0.f; }
       }
+      if (KEYED) {
+        for (int e = tid - NC; e < CH * Kp; e += LS_PREP) {
+          if (e % Kp >= K) { sm[KEYS_AT + e] = 0.f; sm[BUF + KEYS_AT + e] = 0.f; }
+        }
+      }
       ls_prep_barrier();
     }
     prepare(0, sm);
@@ -317,8 +365,9 @@ linear_state_kernel(const LsArgs a) {
     const int n = min(CH, qlen - c * CH);
     // one token: the state's columns walk on, `out` takes this lane's share of the read-out
     auto token = [&](int t, float& out) {
-      const float g = sg[t];
+      const float g = KEYED ? 1.0f : sg[t];
       float kk[KR], qq[KR];
+      const float* sd = buf + KEYS_AT;
 #pragma unroll
       for (int m = 0; m < M; ++m) {
         const float4 k4 = *reinterpret_cast<const float4*>(sk + t * Kp + 4 * (lane + LS_LANES * m));
@@ -347,6 +396,10 @@ linear_state_kernel(const LsArgs a) {
       float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
 #pragma unroll
       for (int m = 0; m < M; ++m) {
+        if (KEYED) {
+          const float4 d4 = *reinterpret_cast<const float4*>(sd + t * Kp + 4 * (lane + LS_LANES * m));
+          S[4 * m] *= d4.x; S[4 * m + 1] *= d4.y; S[4 * m + 2] *= d4.z; S[4 * m + 3] *= d4.w;
+        }
         S[4 * m] = fmaf(kk[4 * m], u, g * S[4 * m]);
         S[4 * m + 1] = fmaf(kk[4 * m + 1], u, g * S[4 * m + 1]);
         S[4 * m + 2] = fmaf(kk[4 * m + 2], u, g * S[4 * m + 2]);
@@ -402,41 +455,53 @@ int ls_sm_count() {
   return n[dev];
 }
 
-template <typename T, int KR, int COLS, bool ROT>
+template <typename T, int KR, int COLS, bool ROT, bool KEYED>
 cudaError_t ls_launch(const LsArgs& a, int n_seqs, bool delta, bool walk, cudaStream_t stream) {
   constexpr int CH = LsChunk<KR>::value;
-  const size_t smem = 2 * (size_t)(2 * CH * KR * LS_LANES + 2 * CH * COLS + 2 * CH) * sizeof(float);
+  const size_t smem = 2 * (size_t)((KEYED ? 3 : 2) * CH * KR * LS_LANES + 2 * CH * COLS + 2 * CH) * sizeof(float);
   const dim3 grid(a.heads, n_seqs, (a.V + COLS - 1) / COLS), block(COLS * LS_LANES + LS_PREP);
-  if constexpr (ROT) {
-    return walk ? gi::launch(linear_state_kernel<T, KR, COLS, false, true, true>, grid, block, smem, stream, a)
-                : gi::launch(linear_state_kernel<T, KR, COLS, false, false, true>, grid, block, smem, stream, a);
+  if constexpr (KEYED) {
+    auto kern = walk ? linear_state_kernel<T, KR, COLS, false, true, false, true> : linear_state_kernel<T, KR, COLS, false, false, false, true>;
+    if (smem > 48 * 1024) {
+      static bool configured[2][gi::MAX_DEVICES_SEEN] = {};
+      int dev;
+      if (gi::unconfigured_here(configured[walk ? 1 : 0], &dev)) {
+        const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return e;
+        if (dev >= 0) configured[walk ? 1 : 0][dev] = true;
+      }
+    }
+    return gi::launch(kern, grid, block, smem, stream, a);
+  } else if constexpr (ROT) {
+    return walk ? gi::launch(linear_state_kernel<T, KR, COLS, false, true, true, false>, grid, block, smem, stream, a)
+                : gi::launch(linear_state_kernel<T, KR, COLS, false, false, true, false>, grid, block, smem, stream, a);
   } else {
     if (walk)
-      return delta ? gi::launch(linear_state_kernel<T, KR, COLS, true, true, false>, grid, block, smem, stream, a)
-                   : gi::launch(linear_state_kernel<T, KR, COLS, false, true, false>, grid, block, smem, stream, a);
-    return delta ? gi::launch(linear_state_kernel<T, KR, COLS, true, false, false>, grid, block, smem, stream, a)
-                 : gi::launch(linear_state_kernel<T, KR, COLS, false, false, false>, grid, block, smem, stream, a);
+      return delta ? gi::launch(linear_state_kernel<T, KR, COLS, true, true, false, false>, grid, block, smem, stream, a)
+                   : gi::launch(linear_state_kernel<T, KR, COLS, false, true, false, false>, grid, block, smem, stream, a);
+    return delta ? gi::launch(linear_state_kernel<T, KR, COLS, true, false, false, false>, grid, block, smem, stream, a)
+                 : gi::launch(linear_state_kernel<T, KR, COLS, false, false, false, false>, grid, block, smem, stream, a);
   }
 }
 
-template <typename T, int KR, bool ROT>
+template <typename T, int KR, bool ROT, bool KEYED>
 cudaError_t ls_pick_tile(const LsArgs& a, int n_seqs, bool delta, bool walk, cudaStream_t stream) {
   // the widest tile that still gives every SM a block: with fewer blocks than SMs the token-by-token walk, whose length a
   // block cannot shorten, runs on a part of the device only
   const long per = (long)a.heads * n_seqs, sms = ls_sm_count();
-  if (per * ((a.V + 31) / 32) >= sms || a.V <= 8) return ls_launch<T, KR, 32, ROT>(a, n_seqs, delta, walk, stream);
-  if (per * ((a.V + 15) / 16) >= sms) return ls_launch<T, KR, 16, ROT>(a, n_seqs, delta, walk, stream);
-  return ls_launch<T, KR, 8, ROT>(a, n_seqs, delta, walk, stream);
+  if (per * ((a.V + 31) / 32) >= sms || a.V <= 8) return ls_launch<T, KR, 32, ROT, KEYED>(a, n_seqs, delta, walk, stream);
+  if (per * ((a.V + 15) / 16) >= sms) return ls_launch<T, KR, 16, ROT, KEYED>(a, n_seqs, delta, walk, stream);
+  return ls_launch<T, KR, 8, ROT, KEYED>(a, n_seqs, delta, walk, stream);
 }
 
 // What every entry point checks and fills in alike (the pointers and sizes are set).
-template <bool ROT>
+template <bool ROT, bool KEYED = false>
 int ls_run(LsArgs& a, int dtype, int n_seqs, int delta, int n_tokens, void* stream) {
   const int K = a.K, V = a.V;
   if (a.heads <= 0 || a.qk_heads <= 0 || a.heads % a.qk_heads || K <= 0 || V <= 0)
     return gi::fail(GI_ERR_ARG, "linear_state: bad sizes (heads %d, query/key heads %d, keys %d, values %d)", a.heads, a.qk_heads, K, V);
   if (K > 32 * LS_LANES) return gi::fail(GI_ERR_UNSUPPORTED, "linear_state: keys of %d numbers (at most %d)", K, 32 * LS_LANES);
-  if (!a.o || !a.q || !a.k || !a.v || (!a.decay_c && !a.g_direct) || !a.state || !a.cu_seqlens || !a.seq_slots)
+  if (!a.o || !a.q || !a.k || !a.v || (!a.decay_c && !a.g_direct && !a.g_key) || !a.state || !a.cu_seqlens || !a.seq_slots)
     return gi::fail(GI_ERR_ARG, "linear_state: a missing pointer");
   if (a.state_ld < (long)a.heads * K * V)
     return gi::fail(GI_ERR_ARG, "linear_state: state rows of %ld floats, wanted %ld", a.state_ld, (long)a.heads * K * V);
@@ -453,10 +518,10 @@ int ls_run(LsArgs& a, int dtype, int n_seqs, int delta, int n_tokens, void* stre
   const bool walk = n_tokens <= 0 || n_tokens > n_seqs;
   cudaError_t e = cudaSuccess;
   GI_DISPATCH_DTYPE(dtype, T, {
-    if (K <= 4 * LS_LANES) e = ls_pick_tile<T, 4, ROT>(a, n_seqs, delta != 0, walk, (cudaStream_t)stream);
-    else if (K <= 8 * LS_LANES) e = ls_pick_tile<T, 8, ROT>(a, n_seqs, delta != 0, walk, (cudaStream_t)stream);
-    else if (K <= 16 * LS_LANES) e = ls_pick_tile<T, 16, ROT>(a, n_seqs, delta != 0, walk, (cudaStream_t)stream);
-    else e = ls_pick_tile<T, 32, ROT>(a, n_seqs, delta != 0, walk, (cudaStream_t)stream);
+    if (K <= 4 * LS_LANES) e = ls_pick_tile<T, 4, ROT, KEYED>(a, n_seqs, delta != 0, walk, (cudaStream_t)stream);
+    else if (K <= 8 * LS_LANES) e = ls_pick_tile<T, 8, ROT, KEYED>(a, n_seqs, delta != 0, walk, (cudaStream_t)stream);
+    else if (K <= 16 * LS_LANES) e = ls_pick_tile<T, 16, ROT, KEYED>(a, n_seqs, delta != 0, walk, (cudaStream_t)stream);
+    else e = ls_pick_tile<T, 32, ROT, KEYED>(a, n_seqs, delta != 0, walk, (cudaStream_t)stream);
   });
   return gi::check(e, "linear_state");
 }

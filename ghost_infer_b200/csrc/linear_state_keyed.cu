@@ -1,0 +1,77 @@
+// Linear attention whose state decays by a number per token and key channel ("gated linear attention"): the recurrence of
+// linear_state.cuh in that form, and the kernel that makes the decays.
+//
+//  * key_decays:  g[t][c] = sigmoid(z)^(1 / tau), z = sum_r low[t][r] up[r][c] + b[c]: the second of two matrices, its bias and
+//                 the root in one pass, 32-bit (low: rows of the projection in the activation type).
+#include "linear_state.cuh"
+
+namespace {
+
+constexpr int KD_TOK = 8;      // tokens per block
+constexpr int KD_RANK = 64;    // numbers of a row in shared memory at a time
+
+// grid (token tiles, channel tiles of 256): a thread takes one channel of eight tokens
+template <typename T>
+__global__ void __launch_bounds__(256)
+key_decays_kernel(float* __restrict__ g, const T* low, long ldl, const float* __restrict__ up, const float* __restrict__ b, int n_tokens,
+                  int rank, int channels, float inv_tau) {
+  __shared__ float sl[KD_TOK][KD_RANK];
+  gi::pdl_prologue();
+  const int t0 = blockIdx.x * KD_TOK, n = min(KD_TOK, n_tokens - t0);
+  const int c = blockIdx.y * 256 + threadIdx.x;
+  float z[KD_TOK];
+  const float bias = c < channels ? b[c] : 0.f;
+#pragma unroll
+  for (int t = 0; t < KD_TOK; ++t) z[t] = bias;
+  for (int r0 = 0; r0 < rank; r0 += KD_RANK) {
+    const int nr = min(KD_RANK, rank - r0);
+    __syncthreads();
+    for (int i = threadIdx.x; i < KD_TOK * KD_RANK; i += 256) {
+      const int t = i / KD_RANK, r = i % KD_RANK;
+      sl[t][r] = (t < n && r < nr) ? gi::ldf(low + (size_t)(t0 + t) * ldl + r0 + r) : 0.f;
+    }
+    __syncthreads();
+    if (c < channels) {
+      for (int r = 0; r < nr; ++r) {
+        const float u = up[(size_t)(r0 + r) * channels + c];
+#pragma unroll
+        for (int t = 0; t < KD_TOK; ++t) z[t] = fmaf(sl[t][r], u, z[t]);
+      }
+    }
+  }
+  if (c >= channels) return;
+#pragma unroll
+  for (int t = 0; t < KD_TOK; ++t)
+    if (t < n) g[(size_t)(t0 + t) * channels + c] = expf(-inv_tau * ls_softplus(-z[t]));      // sigmoid(z) = exp(-softplus(-z))
+}
+
+}  // namespace
+
+extern "C" int gi_key_decays(float* g, const void* low, long ldl, int dtype, const float* up, const float* b, int n_tokens, int rank, int channels,
+                             float tau, void* stream) {
+  if (n_tokens <= 0) return GI_OK;
+  if (rank <= 0 || channels <= 0 || !(tau > 0.f)) return gi::fail(GI_ERR_ARG, "key_decays: bad sizes (rank %d, channels %d, tau %g)", rank, channels, tau);
+  if (!g || !low || !up || !b) return gi::fail(GI_ERR_ARG, "key_decays: a missing pointer");
+  const dim3 grid((n_tokens + KD_TOK - 1) / KD_TOK, (channels + 255) / 256);
+  if (grid.y > 65535) return gi::fail(GI_ERR_UNSUPPORTED, "key_decays: too many channels");
+  cudaError_t e = cudaSuccess;
+  GI_DISPATCH_DTYPE(dtype, T,
+      e = gi::launch(key_decays_kernel<T>, grid, dim3(256), 0, (cudaStream_t)stream, g, (const T*)low, ldl, up, b, n_tokens, rank, channels, 1.0f / tau));
+  return gi::check(e, "key_decays");
+}
+
+extern "C" int gi_linear_state_keyed(float* o, const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, int dtype,
+                                     const float* decay, float q_scale, float* state, long state_ld, int state_rows,
+                                     const int* cu_seqlens, const int* seq_slots, int n_seqs, int heads, int K, int V, int n_tokens,
+                                     void* stream) {
+  if (n_seqs <= 0) return GI_OK;
+  if (decay == nullptr || ((uintptr_t)decay & 15)) return gi::fail(GI_ERR_ARG, "linear_state: the decays per key must start on a 16-byte boundary");
+  LsArgs a = {};
+  a.o = o; a.q = q; a.k = k; a.v = v;
+  a.ldq = ldq; a.ldk = ldk; a.ldv = ldv;
+  a.g_key = decay; a.state = state; a.state_ld = state_ld; a.state_rows = state_rows;
+  a.cu_seqlens = cu_seqlens; a.seq_slots = seq_slots;
+  a.heads = heads; a.qk_heads = heads; a.K = K; a.V = V;
+  a.q_scale = q_scale; a.k_scale = 1.0f;
+  return ls_run<false, true>(a, dtype, n_seqs, 0, n_tokens, stream);
+}

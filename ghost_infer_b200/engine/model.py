@@ -49,6 +49,7 @@ class Layer:
         if mixer_norm is None and mixer is None and ffn_norm is None and ffn is None and not extra:
             raise ValueError(f"layer {index} has no parts")
         self.block = lookup("block", spec.block)(mixer_norm, mixer, ffn_norm, ffn, **extra)
+        self.block.params = dict(getattr(spec, "block_params", {}))
 
     def weights(self) -> List[WeightSpec]:
         out: List[WeightSpec] = []

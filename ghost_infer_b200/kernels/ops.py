@@ -142,6 +142,11 @@ def _bind():
         "gi_latent_prepare_q": [P, P, I, L, P, P, I, F, P, I, P, P, P, I, P, I, I, I, I, I, P, L, P, L, I, I, P],
         "gi_attn_latent_tc_ex": [P, L, P, P, P, L, P, P, I, P, P, P, P, I, I, I, I, I, F, I, I, I, P, P, L, P],
         "gi_linear_state_rot": [P, P, L, P, L, P, L, I, P, P, I, I, F, P, L, I, P, P, I, I, I, I, I, P],
+        "gi_join_rows": [P, P, F, P, I, P, I, I, I, F, SettleT, P],
+        "gi_map_prepare": [P, L, I, P, L, P, I, P, L, I, I, P, I, I, P, P, P, I, P, P, I, I, I, I, I, P],
+        "gi_map_difference": [P, P, I, I, I, I, F, F, F, P],
+        "gi_key_decays": [P, P, L, I, P, P, I, I, I, F, P],
+        "gi_linear_state_keyed": [P, P, L, P, L, P, L, I, P, F, P, L, I, P, P, I, I, I, I, I, P],
         "gi_attn_decode_generic_ex3": [P, L, P, P, P, L, I, P, P, P, I, P, P, I, I, I, I, F, I, I, I, I, F, P, I, L, I, P],
     }
     for name, argtypes in sigs.items():
@@ -2563,4 +2568,128 @@ def linear_state_rot(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: t
         decay.data_ptr(), table.data_ptr() if half else None, half, int(bool(adjacent)), float(k_scale), state.data_ptr(),
         state.stride(0), state.shape[0], _i32(step.cu_seqlens, "cu_seqlens"), _i32(step.seq_slots, "slots"), step.n_seqs, heads,
         key_dim, v_dim, int(n), _stream()))
+    return o
+
+
+# ---- a stream joined once a layer, heads that are the difference of two maps, decays per key channel ------------------------
+def join_rows(x: torch.Tensor, y: torch.Tensor, scale: float, read=None) -> Optional[torch.Tensor]:
+    """x += scale * y (float32 rows), y zeroed; returns, where `read` (weight, eps, dtype) is given, the rows' RMS norm.  Partial
+    sums that a deferred product left for y are added on the way."""
+    lib = _bind()
+    settle(x)
+    for t, what in ((x, "stream rows"), (y, "sublayer rows")):
+        _cuda(t, what, settles=t is y)
+        if t.dtype != torch.float32 or t.shape != x.shape or not t.is_contiguous():
+            raise KernelError(f"{what} must be contiguous float32 {tuple(x.shape)}, got {t.dtype} {tuple(t.shape)}")
+    n, d = x.shape
+    h = w = None
+    eps = 0.0
+    if read is not None:
+        w, eps, dtype = read
+        if w.numel() != d or not w.is_contiguous():
+            raise KernelError(f"the norm's weight has {w.numel()} values, the rows are {d} wide")
+        h = torch.empty((n, d), dtype=dtype, device=x.device)
+    rec = SettleT(None, None, None, None, 0)
+    if has_pending(y):
+        threads = 1024 if d >= 4096 else (512 if d >= 2048 else 256)
+        aligned = all(t is None or t.data_ptr() % 16 == 0 for t in (x, y, w))
+        if y.__dict__["_gi_pending"][1] or d % 4 or d > 16 * threads or not aligned:
+            settle(y)
+        else:
+            rec = _take_pending(y)[0]
+    _check(lib, lib.gi_join_rows(x.data_ptr(), y.data_ptr(), float(scale), h.data_ptr() if h is not None else None,
+                                 _dt(h, "normed rows") if h is not None else F32, w.data_ptr() if w is not None else None,
+                                 _dt(w, "norm weight") if w is not None else F32, n, d, float(eps), rec, _stream()))
+    return h
+
+
+def map_prepare(rows: torch.Tensor, out_dtype: torch.dtype, conv: Optional[torch.Tensor], state: Optional[torch.Tensor],
+                table: Optional[torch.Tensor], rot_dims: int, adjacent: bool, step, memory, n_heads: int, n_kv: int, dim: int,
+                v_dim: int) -> torch.Tensor:
+    """Float32 projection rows [q: heads x 2 x dim | k: kv heads x 2 x dim | v] to queries [tokens, heads * 2 * 2 dim] (each of a
+    head's two maps a row of 2 dim numbers with zeros in the other's place), with keys (both maps side by side) and values written
+    to `memory`'s pages.  `conv` float32 [taps, channels] or None: the causal convolution every channel passes first, whose older
+    inputs live in `state` ([slots + 1, (taps - 1) * channels] float32), which takes the step's last inputs."""
+    lib = _bind()
+    _cuda(rows, "projection rows")
+    n = rows.shape[0]
+    n2 = 2 * dim
+    channels = (n_heads + n_kv) * n2 + n_kv * v_dim
+    if rows.dtype != torch.float32 or rows.dim() != 2 or rows.stride(1) != 1 or rows.shape[1] < channels:
+        raise KernelError(f"map_prepare: float32 projection rows of {channels} numbers are wanted")
+    taps = 0 if conv is None else conv.shape[0]
+    if conv is not None and (conv.dtype != torch.float32 or tuple(conv.shape) != (taps, channels) or not conv.is_contiguous() or not conv.is_cuda):
+        raise KernelError(f"map_prepare: the convolution's taps must be contiguous float32 [taps, {channels}]")
+    sp, sld, srows = _conv_state(state, taps, channels)
+    if memory.k is None or not memory.writes or memory.k.dtype != out_dtype or memory.v is None or memory.v.dtype != out_dtype:
+        raise KernelError("map_prepare: keys and values need a cache of the step's type that this entry writes")
+    if (tuple(memory.k.shape[1:]) != (n_kv, 64, n2) or tuple(memory.v.shape[1:]) != (n_kv, 64, v_dim)
+            or not memory.k.is_contiguous() or not memory.v.is_contiguous()):
+        raise KernelError(f"cache pages must be contiguous [pages, {n_kv}, 64, {n2}] and [.., {v_dim}]")
+    half = rot_dims // 2
+    if half and (table is None or table.dtype != torch.float32 or tuple(table.shape) != (n, half, 2) or not table.is_contiguous()):
+        raise KernelError(f"the table of angles must be contiguous float32 [{n}, {half}, 2]")
+    q = torch.empty((n, n_heads * 2 * n2), dtype=out_dtype, device=rows.device)
+    bt = memory.block_table
+    one_each = bool(step.is_decode)
+    _check(lib, lib.gi_map_prepare(
+        q.data_ptr(), q.stride(0), _DT[out_dtype], rows.data_ptr(), rows.stride(0), conv.data_ptr() if taps else None, taps, sp, sld,
+        srows, int(one_each), table.data_ptr() if half else None, half, int(bool(adjacent)), _i32(step.positions, "positions"),
+        _i32(step.token_slots, "slots"), _i32(bt, "block table"), bt.shape[1], memory.k.data_ptr(), memory.v.data_ptr(), n, n_heads,
+        n_kv, dim, v_dim, _stream()))
+    if taps > 1 and not one_each:
+        _check(lib, lib.gi_mamba2_conv_update(rows.data_ptr(), F32, rows.stride(0), sp, sld, srows, _i32(step.cu_seqlens, "cu_seqlens"),
+                                              _i32(step.seq_slots, "slots"), step.n_seqs, 0, channels, taps, 0, _stream()))
+    return q
+
+
+def map_difference(a: torch.Tensor, n_heads: int, v_dim: int, weight: float, factor: float, eps: float) -> torch.Tensor:
+    """Rows [heads][2 maps][values] to rows [heads][values]: v = first - weight * second; factor * v / sqrt(mean(v^2) + eps)."""
+    lib = _bind()
+    _cuda(a, "attention output")
+    n = a.shape[0]
+    if not a.is_contiguous() or a.shape[1] != 2 * n_heads * v_dim:
+        raise KernelError("map_difference: contiguous rows of two maps a head are wanted")
+    out = torch.empty((n, n_heads * v_dim), dtype=a.dtype, device=a.device)
+    _check(lib, lib.gi_map_difference(out.data_ptr(), a.data_ptr(), _dt(a, "attention output"), n, n_heads, v_dim, float(weight),
+                                      float(factor), float(eps), _stream()))
+    return out
+
+
+def key_decays(low: torch.Tensor, up: torch.Tensor, bias: torch.Tensor, tau: float) -> torch.Tensor:
+    """sigmoid(low @ up + bias)^(1 / tau), float32 [tokens, channels]; `low` may be a view of wider rows, `up` float32 [rank, channels]."""
+    lib = _bind()
+    _cuda(low, "decay rows")
+    rank, channels = up.shape
+    if low.dim() != 2 or low.shape[1] != rank or low.stride(1) != 1:
+        raise KernelError(f"decay rows must be [tokens, {rank}], got {tuple(low.shape)}")
+    for t, size in ((up, rank * channels), (bias, channels)):
+        if t.dtype != torch.float32 or t.numel() != size or not t.is_contiguous() or not t.is_cuda:
+            raise KernelError("the decays' matrix and bias must be contiguous float32 on the device")
+    g = torch.empty((low.shape[0], channels), dtype=torch.float32, device=low.device)
+    _check(lib, lib.gi_key_decays(g.data_ptr(), low.data_ptr(), low.stride(0), _dt(low, "decay rows"), up.data_ptr(), bias.data_ptr(),
+                                  low.shape[0], rank, channels, float(tau), _stream()))
+    return g
+
+
+def linear_state_keyed(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, step, heads: int,
+                       key_dim: int, v_dim: int, q_scale: float) -> torch.Tensor:
+    """The recurrence S <- diag(decay_t) S + k_t v_t^T; o_t = S^T (q_scale q_t) with a decay per token and key channel, float32
+    [tokens, heads * key_dim], from and into `state` ([slots + 1, >= heads * key_dim * v_dim] float32).  Returns float32
+    [tokens, heads * v_dim]."""
+    lib = _bind()
+    n = q.shape[0]
+    for t, what, width in ((q, "queries", heads * key_dim), (k, "keys", heads * key_dim), (v, "values", heads * v_dim)):
+        _cuda(t, what)
+        if t.dtype != q.dtype or tuple(t.shape) != (n, width) or t.stride(1) != 1:
+            raise KernelError(f"{what} must be [{n}, {width}] rows of the queries' type, got {t.dtype} {tuple(t.shape)}")
+    if decay.dtype != torch.float32 or tuple(decay.shape) != (n, heads * key_dim) or not decay.is_contiguous() or not decay.is_cuda:
+        raise KernelError(f"decays must be contiguous float32 [{n}, {heads * key_dim}] on the device")
+    if state is None or state.dtype != torch.float32 or state.dim() != 2 or not state.is_contiguous() or state.shape[1] < heads * key_dim * v_dim:
+        raise KernelError("the recurrence needs its per-sequence state as a contiguous float32 matrix of at least heads x keys x values")
+    o = torch.empty((n, heads * v_dim), dtype=torch.float32, device=q.device)
+    _check(lib, lib.gi_linear_state_keyed(
+        o.data_ptr(), q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), _dt(q, "queries"),
+        decay.data_ptr(), float(q_scale), state.data_ptr(), state.stride(0), state.shape[0], _i32(step.cu_seqlens, "cu_seqlens"),
+        _i32(step.seq_slots, "slots"), step.n_seqs, heads, key_dim, v_dim, int(n), _stream()))
     return o

@@ -45,6 +45,7 @@ class WeightSpec(NamedTuple):
     shape: Tuple[int, ...]
     init: str = "normal"       # how the random-weights mode fills it: "normal" or "ones"
     shared: bool = False       # several parts may name this tensor (one table, read by every layer); it is loaded once
+    free: Tuple[int, ...] = () # axes whose size the weights file decides (`shape` then says what random weights take)
 
 
 @dataclass
@@ -104,6 +105,14 @@ class StreamRead(NamedTuple):
     base: Optional[torch.Tensor] = None
 
 
+class RowRead(NamedTuple):
+    """A norm over whole rows that a pass which holds a whole row of the stream can do on the way: h = x / sqrt(mean(x^2) + eps) *
+    weight, in `dtype`."""
+    weight: torch.Tensor
+    eps: float
+    dtype: torch.dtype
+
+
 class Norm(Part):
     def forward(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         raise NotImplementedError
@@ -114,6 +123,10 @@ class Norm(Part):
 
     def stream_read(self, step) -> Optional[StreamRead]:
         """Element-wise norms can run inside the pass that writes the stream: what that pass has to know.  None: they cannot."""
+        return None
+
+    def row_read(self, step) -> Optional[RowRead]:
+        """RMS norms can run inside a pass that writes whole rows of the stream.  None: this norm cannot."""
         return None
 
 
@@ -185,7 +198,8 @@ class FeedForward(Part):
 
 class Block:
     """An arrangement of one layer's parts: the usual four (any of which an arrangement may lack: None) and whatever
-    else the layer's specification names (`self.extra[name]`)."""
+    else the layer's specification names (`self.extra[name]`).  `params`: the arrangement's own constants."""
+    params: Mapping[str, Any] = {}
 
     def __init__(self, mixer_norm: Optional[Norm] = None, mixer: Optional[Mixer] = None, ffn_norm: Optional[Norm] = None,
                  ffn: Optional[FeedForward] = None, **extra: Part):

@@ -96,3 +96,37 @@ class SandwichResidual(Block):
                        self.ffn_norm if self.ffn is not None else last)
         if self.ffn is not None:
             self._sublayer(x, step, self.ffn_norm, self.extra["ffn_post"], lambda h, y: self.ffn.forward(h, y, step), last)
+
+
+@register("block", "parallel_residual")
+class ParallelResidual(Block):
+    """x += s * (mixer(n(x)) + ffn(n(x))), s = `params["scale"]` (1 unless given): one norm, which both sublayers read.  They add
+    into 32-bit rows of their own; one pass joins those to the stream (with whatever partial sums the last product left in them),
+    zeroes them for the next layer and, where the next reader of the stream is a norm that says so (`row_read`), does that norm
+    on the way.  Stream, norms and sums are 32-bit."""
+
+    def first_reader(self):
+        return self.mixer_norm
+
+    def forward(self, x, step, memory) -> None:
+        if x.is_cuda and not getattr(self.mixer_norm, "settles_pending", False):
+            ops.settle(x)
+        h = self.mixer_norm.forward(x)
+        key = ("sublayer rows", tuple(x.shape))
+        y = step.shared.get(key)
+        if y is None:
+            y = step.shared[key] = ops.as_carrier(torch.zeros(x.shape, dtype=torch.float32, device=x.device))
+        runs = [lambda: self.mixer.forward(h, y, step, memory)] if self.mixer is not None else []
+        if self.ffn is not None:
+            runs.append(lambda: self.ffn.forward(h, y, step))
+        for run in runs[:-1]:
+            run()
+        if runs:
+            with ops.defer_into(y):       # nothing but the join reads the rows after the last product
+                runs[-1]()
+        reader = step.next_reader
+        read = reader.row_read(step) if reader is not None and hasattr(reader, "row_read") else None
+        with ops.bucket("norm"):
+            nxt = ops.join_rows(x, y, float(self.params.get("scale", 1.0)), read)
+        if nxt is not None:
+            ops.hand_on(x, reader, nxt)

@@ -8,10 +8,11 @@ values of `v_head_dim` numbers:
                that all heads share (before the rotation);  `v_norm`: every head of v is divided by its root mean square, and
                cached so
     the first `rotary.dims` numbers of every head of q and k turn by position * base^(-2i / dims), pairs (i, i + dims / 2)
-               (`rotary.pairing` "half") or (2i, 2i + 1) ("adjacent"); the rest of a head passes
+               (`rotary.pairing` "half") or (2i, 2i + 1) ("adjacent"), the angles scaled by `rotary.scaling` where it is
+               given; the rest of a head passes
     score = (q . k) * scale;  position i sees j <= i with i - j < `window` or j < `keep_first` (kept positions keep their
-               true positions); softmax in 32-bit, with `sink` a learned number per head whose exponential joins the
-               denominator without key or value
+               true positions); softmax in 32-bit, with `sink` True a learned number per head whose exponential joins
+               the denominator without key or value, with `sink` "zero" a one that joins it (no tensor)
     `head_gate`: head a's output is multiplied by sigmoid(Wg h)_a, one number per head
     residual += Wo (heads) (+ bo)
 
@@ -54,7 +55,11 @@ class HeadNormedAttention(Mixer):
         self.bias = bool(params.get("bias", False))
         self.qk_norm = bool(params.get("qk_norm", False))
         self.v_norm = bool(params.get("v_norm", False))
-        self.has_sink = bool(params.get("sink", False))
+        sink = params.get("sink", False)
+        if sink not in (False, None, True, "zero"):
+            raise ValueError(f"sink must be False, True or \"zero\", got {sink!r}")
+        self.zero_sink = sink == "zero"
+        self.has_sink = bool(sink) and not self.zero_sink            # a learned one, with a tensor
         self.head_gate = bool(params.get("head_gate", False))
         self.eps = float(params.get("eps", 1e-6))
         self.borrows_kv = bool(params.get("borrows_kv", False))
@@ -69,7 +74,7 @@ class HeadNormedAttention(Mixer):
         if rot is not None and int(rot["dims"]) > 0:
             self.rot_dims = int(rot["dims"])
             self.rotary = Rotary({"head_dim": self.head_dim, "rotary_dim": self.rot_dims, "theta": float(rot["base"]),
-                                  "pairing": rot.get("pairing", "half")}, prefix)
+                                  "pairing": rot.get("pairing", "half"), "scaling": rot.get("scaling")}, prefix)
         self.adjacent = self.rotary is not None and self.rotary.pairing == "adjacent"
         self.q_dim, self.k_dim, self.v_width = self.n_heads * self.head_dim, self.n_kv * self.head_dim, self.n_kv * self.v_dim
         base = str(params.get("base", "mix."))
@@ -123,6 +128,8 @@ class HeadNormedAttention(Mixer):
         self.b_o = f32(n["o.b"]) if self.bias else None
         self.norm_w = (f32(n["q.norm"]), f32(n["k.norm"]) if kv else None) if self.qk_norm else (None, None)
         self.sinks = f32(n["sink"]) if self.has_sink else None
+        if self.zero_sink:
+            self.sinks = torch.zeros((self.n_heads,), dtype=torch.float32, device=rt.device)
         if self.rotary is not None:
             self.rotary.bind(tensors, rt)
 

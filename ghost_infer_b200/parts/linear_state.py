@@ -1,6 +1,7 @@
-"""Mixers that carry a matrix of state per head from token to token: a gated delta rule, decayed linear attention, retention.
+"""Mixers that carry a matrix of state per head from token to token: a gated delta rule, decayed linear attention, retention, gated
+linear attention.
 
-Both walk, per head, S (a key_dim x v_dim matrix of 32-bit numbers, zero when a sequence starts):
+All walk, per head, S (a key_dim x v_dim matrix of 32-bit numbers, zero when a sequence starts):
 
     S <- g_t S;   u_t = v_t (or, delta rule: beta_t (v_t - S^T k_t));   S <- S + k_t u_t^T;   o_t = S^T q_t
 
@@ -20,8 +21,13 @@ sigmoid(Wg h), and projected: residual += Wo (...).  Per sequence: S.
 (`decay`); each head's o is divided by its root mean square over v_dim (eps, no weight), the heads side by side are multiplied
 by silu(Wg h), and projected: residual += Wo (...).  Per sequence: S.
 
+"gated_linear_attention": q = Wq h, times key_dim^(-1/2), and k = Wk h (heads of key_dim), v = Wv h (heads of v_dim), no
+activation; the decay is one number per key channel and token, S <- diag(g_t) S, g = sigmoid(Wa2 (Wa1 h) + b)^(1 / `tau`)
+(heads * key_dim of them; the width between Wa1 and Wa2 is the tensors'); each head's o is divided by its root mean square over
+v_dim (eps), times a weight of v_dim shared by the heads, times silu(Wg h), and projected: residual += Wo (...).  Per sequence: S.
+
 The recurrence, decays, gates of the recurrence, unit norms and output norms are 32-bit in both precisions.
-Tensor names: prefix + `base` + {q, q.conv, k, k.conv, v, v.conv, b, a, A_log, dt_bias, norm, g, o} (`base` "mix.").
+Tensor names: prefix + `base` + {q, q.conv, k, k.conv, v, v.conv, b, a, A_log, dt_bias, a1, a2, a2.b, norm, g, o} (`base` "mix.").
 """
 from __future__ import annotations
 
@@ -203,5 +209,65 @@ class Retention(Mixer):
                                      self.key_dim, self.v_dim, self.decay_dev, table, self.rot, self.adjacent, self.key_dim ** -0.5)
         with ops.bucket("gated norm"):
             y = ops.norm_gate(o, proj[:, 2 * qk + vw:2 * qk + 2 * vw], None, self.v_dim, self.eps, "silu", self.rt.dtype)
+        with ops.bucket("out matmul"):
+            linear(y, self.w_o, out=residual, accumulate=True)
+
+
+@register("mixer", "gated_linear_attention")
+class GatedLinearAttention(Mixer):
+    RANK = 16          # the width between the decay's two matrices where no file says another (random weights)
+
+    def __init__(self, params, prefix=""):
+        super().__init__(params, prefix)
+        self.hidden = int(params["hidden_size"])
+        self.heads = int(params["heads"])
+        self.key_dim = int(params["key_dim"])
+        self.v_dim = int(params["v_dim"])
+        self.tau = float(params["tau"])
+        self.eps = float(params["eps"])
+        self.rank = int(params.get("rank") or self.RANK)
+        if not self.tau > 0:
+            raise ValueError(f"the decays' root must be positive, got {self.tau}")
+        self.qk_width, self.v_width = self.heads * self.key_dim, self.heads * self.v_dim
+        base = str(params.get("base", "mix."))
+        self.names = {k: self.tensor_name(k, base + k) for k in ("q", "k", "v", "g", "o", "norm", "a1", "a2", "a2.b")}
+
+    def weights(self) -> List[WeightSpec]:
+        n, d = self.names, self.hidden
+        return [WeightSpec(n["q"], (self.qk_width, d)), WeightSpec(n["k"], (self.qk_width, d)), WeightSpec(n["v"], (self.v_width, d)),
+                WeightSpec(n["g"], (self.v_width, d)), WeightSpec(n["o"], (d, self.v_width)), WeightSpec(n["norm"], (self.v_dim,), "ones"),
+                WeightSpec(n["a1"], (self.rank, d), free=(0,)), WeightSpec(n["a2"], (self.qk_width, self.rank), free=(1,)),
+                WeightSpec(n["a2.b"], (self.qk_width,))]
+
+    def state_request(self) -> Optional[StateRequest]:
+        return StateRequest((self.heads * self.key_dim * self.v_dim,), torch.float32)
+
+    def bind(self, tensors, rt) -> None:
+        super().bind(tensors, rt)
+        n = self.names
+        a1, a2 = tensors[n["a1"]], tensors[n["a2"]]
+        self.rank = int(a1.shape[0])
+        if int(a2.shape[1]) != self.rank:
+            raise ValueError(f"{n['a1']} has {self.rank} rows, {n['a2']} takes {int(a2.shape[1])}")
+        # one product: [q | k | v | gate | what the decays are made of]
+        self.w_in = stack_rows([rt.place(tensors[n[k]]) for k in ("q", "k", "v", "g", "a1")])
+        self.w_o = rt.place(tensors[n["o"]])
+        # what makes the decays and the norm enters 32-bit arithmetic: kept as 32-bit values (a2 with its outputs side by side)
+        f32 = lambda t: t.to(device=rt.device, dtype=torch.float32).contiguous()
+        self.a2_t, self.a2_b, self.norm_w = f32(a2.to(torch.float32).t()), f32(tensors[n["a2.b"]]), f32(tensors[n["norm"]])
+
+    def forward(self, h, residual, step, memory) -> None:
+        if memory.state is None:
+            raise RuntimeError("linear attention was given no per-sequence state")
+        qk, vw = self.qk_width, self.v_width
+        g0 = 2 * qk + vw
+        with ops.bucket("qkv matmul"):
+            proj = linear(h, self.w_in, out_dtype=self.rt.dtype)
+        with ops.bucket("scan"):
+            keep = ops.key_decays(proj[:, g0 + vw:g0 + vw + self.rank], self.a2_t, self.a2_b, self.tau)
+            o = ops.linear_state_keyed(proj[:, :qk], proj[:, qk:2 * qk], proj[:, 2 * qk:g0], keep, memory.state, step, self.heads,
+                                       self.key_dim, self.v_dim, self.key_dim ** -0.5)
+        with ops.bucket("gated norm"):
+            y = ops.norm_gate(o, proj[:, g0:g0 + vw], self.norm_w, self.v_dim, self.eps, "silu", self.rt.dtype)
         with ops.bucket("out matmul"):
             linear(y, self.w_o, out=residual, accumulate=True)

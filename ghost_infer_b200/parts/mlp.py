@@ -6,8 +6,9 @@ path packs them (src/quant.rs:1135-1154, src/model.rs:1133-1147, src/cuda.rs:923
 Tensor names: prefix + "mlp.{gate,up,down}_proj.weight" unless `params["tensor_names"]` gives others for the
 keys "gate", "up", "down".
 
-The same layer with another activation in place of silu (`params["activation"]`: "silu", the default, or
-"gelu_tanh", 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3)))) is registered as "gated_mlp".
+The same layer with another activation in place of silu (`params["activation"]`: "silu", the default,
+"gelu_tanh", 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))), or "clamped": with g = min(Wgate h, `limit`) and
+u = clamp(Wup h, -`limit`, `limit`) the hidden value is g sigmoid(`alpha` g) (u + 1)) is registered as "gated_mlp".
 
 "mlp": the ungated layer residual += Wdown act(Wup h + b_up) + b_down, with `activation` "relu2" (relu(z)^2) or "gelu"
 (0.5 z (1 + erf(z / sqrt 2)), without biases) and, with
@@ -34,8 +35,13 @@ class SwiGlu(FeedForward):
         self.hidden = int(params["hidden_size"])
         self.inter = int(params["intermediate_size"])
         self.activation = str(params.get("activation", "silu"))
-        if self.activation not in ("silu", "gelu_tanh"):
-            raise ValueError(f"unknown activation \"{self.activation}\" (silu, gelu_tanh)")
+        if self.activation not in ("silu", "gelu_tanh", "clamped"):
+            raise ValueError(f"unknown activation \"{self.activation}\" (silu, gelu_tanh, clamped)")
+        self.limit = self.alpha = 0.0
+        if self.activation == "clamped":
+            self.limit, self.alpha = float(params["limit"]), float(params["alpha"])
+            if not self.limit > 0:
+                raise ValueError(f"the clamped feed-forward needs a positive limit, got {self.limit}")
         self.names = {k: self.tensor_name(k, f"mlp.{k}_proj.weight") for k in ("gate", "up", "down")}
 
     def weights(self) -> List[WeightSpec]:
@@ -63,7 +69,12 @@ class SwiGlu(FeedForward):
 
     def forward(self, h, residual, step) -> None:
         with ops.bucket("ffn matmul"):
-            if self.interleaved:
+            if self.activation == "clamped":
+                if self.interleaved:
+                    act = ops.clamped_glu_interleaved(h, self.w_gate_up, self.limit, self.alpha)
+                else:
+                    act = ops.clamped_glu(linear(h, self.w_gate_up, out_dtype=self.rt.dtype), self.limit, self.alpha)
+            elif self.interleaved:
                 act = ops.swiglu_interleaved(h, self.w_gate_up, self.activation)
             else:
                 gu = linear(h, self.w_gate_up, out_dtype=self.rt.dtype)

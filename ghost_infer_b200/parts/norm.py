@@ -17,7 +17,7 @@ from typing import List, Optional
 import torch
 
 from ..kernels import ops
-from .base import Norm, StreamRead, WeightSpec
+from .base import Norm, RowRead, StreamRead, WeightSpec
 from .registry import register
 
 
@@ -45,7 +45,14 @@ class RmsNorm(Norm):
             self._weight32 = self.weight.to(torch.float32).contiguous()
         return self._weight32
 
+    def row_read(self, step):
+        return RowRead(self.weight, self.eps, self.rt.dtype)
+
     def forward(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+        if rows is None:
+            h = ops.take_handed(x, self)
+            if h is not None and h.dtype == (out_dtype or self.rt.dtype):
+                return h
         with ops.bucket("norm"):
             return ops.rmsnorm(x, self.weight, self.eps, out_dtype or self.rt.dtype, rows=rows)
 

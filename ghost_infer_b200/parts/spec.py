@@ -55,6 +55,7 @@ class LayerSpec:
     mixer_norm_prefix: str = "input_layernorm."            # under `prefix`
     ffn_norm_prefix: str = "post_attention_layernorm."     # under `prefix`
     extra: Tuple[ExtraPart, ...] = ()
+    block_params: Mapping[str, Any] = field(default_factory=dict)      # constants of the arrangement itself (`Block.params`)
 
 
 @dataclass(frozen=True)

@@ -49,7 +49,9 @@ def load_model_tensors(model_dir: str, manifest: Iterable, ignorable: Iterable[s
     for f in files:
         for n in f.names():
             where[n] = f
+    manifest = list(manifest)
     wanted = {w.name: tuple(w.shape) for w in manifest}
+    free = {w.name: tuple(getattr(w, "free", ())) for w in manifest}
     ignorable = set(ignorable)
     missing = [n for n in wanted if n not in where]
     unexpected = sorted(n for n in where if n not in wanted and n not in ignorable)
@@ -57,7 +59,9 @@ def load_model_tensors(model_dir: str, manifest: Iterable, ignorable: Iterable[s
     for n, shape in wanted.items():
         if n in where:
             ent = where[n].entries[n]
-            if tuple(ent.shape) != shape:
+            # an axis whose size the file decides may be of any size but none
+            has = tuple(shape[a] if (a in free[n] and ent.shape[a] > 0) else int(e) for a, e in enumerate(ent.shape)) if len(ent.shape) == len(shape) else tuple(ent.shape)
+            if has != shape:
                 wrong.append(f"{n} is {list(ent.shape)}, the configuration wants {list(shape)}")
             elif ent.dtype not in ("F32", "BF16", "F16", "F64"):
                 wrong.append(f"{n} is stored as {ent.dtype}, not a floating type")
