@@ -268,6 +268,41 @@ VAVUPEL_SIZES = {
 }
 
 
+def _sofopel(width, heads, kv, dim, vdim, chunk, win_heads, win_kv, win_dim, win_vdim, window, keep_first, lin_heads, lin_dim, lin_vdim, ff,
+             vocab, **_):
+    mlp = {"kind": "dense", "ff": ff, "limit": 7.0}
+    maps = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "diff": 0.3, "conv": 4, "mask": {"size": chunk},
+        "rot": {"base": 500000.0, "dims": dim // 2}}}
+    windowed = {"type": "attention_2", "mlp": mlp, "mixer": {
+        "heads": win_heads, "kv_heads": win_kv, "dim": win_dim, "vdim": win_vdim, "scale": win_dim ** -0.5,
+        "mask": {"size": window, "keep_first": keep_first},
+        "rot": {"base": 500000.0, "dims": win_dim, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    linear = {"type": "gla", "mlp": mlp, "mixer": {"heads": lin_heads, "dim": lin_dim, "vdim": lin_vdim, "tau": 16.0}}
+    return {"architecture": "Sofopel", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0}, "residual_mult": 0.5,
+            "loop": {"start": 1, "stop": 3, "times": 2}, "layers": [maps, windowed, linear, windowed]}
+
+
+def _barovik_chunked(z, runs):
+    """Attention in chunks of the same size (capped scores, a sink, no rotation), gated dense feed-forwards of the same width."""
+    c = _barovik(z["width"], z["heads"], z["kv"], 2 * z["dim"], z["vdim"], z["chunk"], z["ff"], 8, 64, 64, 1, 2, 1, 64, 64, z["vocab"], 1)
+    return dict(c, layers=[c["layers"][0]] * runs)
+
+
+# layer sizes of the kind real models have: attention that is the difference of two maps (in chunks), attention in a window that
+# keeps its first positions, and linear attention with a decay per key channel, each with a gated dense feed-forward beside it,
+# the middle two layers run twice (six layer runs).  Beside it, with six layers each: attention in chunks alone, linear attention
+# with windowed attention in turn, and the Llama decoder
+SOFOPEL_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv=4, dim=64, vdim=128, chunk=1024, win_heads=16, win_kv=4, win_dim=128, win_vdim=128, window=1024,
+                  keep_first=64, lin_heads=16, lin_dim=128, lin_vdim=128, ff=8192, vocab=32000, llama_dim=128),
+    "w4096": dict(width=4096, heads=32, kv=8, dim=64, vdim=128, chunk=2048, win_heads=32, win_kv=8, win_dim=128, win_vdim=128, window=2048,
+                  keep_first=128, lin_heads=32, lin_dim=128, lin_vdim=128, ff=14336, vocab=32000, llama_dim=128),
+    "w2048_odd": dict(width=2048, heads=24, kv=4, dim=40, vdim=56, chunk=500, win_heads=20, win_kv=5, win_dim=96, win_vdim=40, window=500,
+                      keep_first=20, lin_heads=12, lin_dim=96, lin_vdim=64, ff=6144, vocab=32000, llama_dim=64),
+}
+
+
 def _barovik_beside(z):
     keys = ("width", "heads", "kv", "dim", "vdim", "chunk", "ff", "ssm_heads", "ssm_dim", "state", "groups", "experts", "top",
             "expert_ff", "shared_ff", "vocab", "pairs")
@@ -275,7 +310,8 @@ def _barovik_beside(z):
 
 
 def measure_hybrid(args):
-    """`--workload barovik` / `--workload navalorn` / `--workload nuzinex` / `--workload torutar` / `--workload vavupel`: prompt and decode throughput of that decoder at a few real layer sizes
+    """`--workload barovik` / `--workload navalorn` / `--workload nuzinex` / `--workload torutar` / `--workload vavupel` /
+    `--workload sofopel`: prompt and decode throughput of that decoder at a few real layer sizes
     (random weights), beside the Llama decoder with the same width, heads, feed-forward width and number of layers (nuzinex:
     beside the hybrid decoder with windowed attention and state-space layers, and the Llama decoder); and the
     device time per kind of operation for one prompt step and one decode step of each.  One JSON line."""
@@ -364,6 +400,8 @@ def measure_hybrid(args):
         sizes, build, label = TORUTAR_SIZES, _torutar, "torutar"
     if args.workload == "vavupel":
         sizes, build, label = VAVUPEL_SIZES, _vavupel, "vavupel"
+    if args.workload == "sofopel":
+        sizes, build, label = SOFOPEL_SIZES, _sofopel, "sofopel"
     names = [n for n in sizes if not args.sizes or n in args.sizes.split(",")]
     for name in names:
         z = sizes[name]
@@ -375,6 +413,11 @@ def measure_hybrid(args):
             out[name]["navalorn_equal_size"] = one(_navalorn_dense(z, 6))
             out[name]["nuzinex_equal_size"] = one(_nuzinex_linear(z, 3))
             out[name]["llama_equal_size"] = one(_llama_like(z["width"], z["heads"], z["kv"], z["dim"], z["ff"], z["vocab"], 6))
+        elif label == "sofopel" and not args.skip_points:
+            out[name]["barovik_equal_size"] = one(_barovik_chunked(z, 6))
+            beside = dict(z, dim=z["win_dim"], heads=z["win_heads"], kv=z["win_kv"], ret_heads=z["lin_heads"], ret_dim=z["lin_dim"], ret_vdim=z["lin_vdim"])
+            out[name]["nuzinex_equal_size"] = one(_nuzinex_linear(beside, 3))
+            out[name]["llama_equal_size"] = one(_llama_like(z["width"], z["heads"], z["kv"], z["llama_dim"], z["ff"], z["vocab"], 6))
         elif not args.skip_points:
             out[name]["llama_equal_size"] = one(_llama_like(z["width"], z["heads"], z["kv"], z["llama_dim"] if latent else z["dim"], z["ff"],
                                                             z["vocab"], 2 * z["pairs"]))
@@ -519,10 +562,10 @@ def main():
     ap.add_argument("--impl", default="ours")
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the named configuration (recorded in config)")
     ap.add_argument("--skip-points", action="store_true")
-    ap.add_argument("--workload", default="8b", choices=["8b", "1b", "3b", "barovik", "navalorn", "nuzinex", "torutar", "vavupel"],
-                    help="8b: the headline; 1b, 3b: the baseline's other workloads; barovik, navalorn, nuzinex, torutar, vavupel: one of the "
+    ap.add_argument("--workload", default="8b", choices=["8b", "1b", "3b", "barovik", "navalorn", "nuzinex", "torutar", "vavupel", "sofopel"],
+                    help="8b: the headline; 1b, 3b: the baseline's other workloads; barovik, navalorn, nuzinex, torutar, vavupel, sofopel: one of the "
                          "other decoders beside the Llama decoder at equal layer sizes (--sizes, --batch, --held)")
-    ap.add_argument("--sizes", default="", help="for --workload barovik / navalorn / nuzinex / torutar / vavupel: which of its sizes to run, with commas (default: all)")
+    ap.add_argument("--sizes", default="", help="for --workload barovik / navalorn / nuzinex / torutar / vavupel / sofopel: which of its sizes to run, with commas (default: all)")
     ap.add_argument("--tune", default="", help="overrides of kernel choices, e.g. small_skinny=0,attn_waves=2")
     ap.add_argument("--only", default="", choices=["", "prefill", "decode", "timeline"],
                     help="run one phase alone and print its time (a short program for a launch list under a profiler; no bench "
@@ -545,7 +588,7 @@ def main():
         for kv in filter(None, args.tune.split(",")):
             k, v = kv.split("=")
             _ops.TUNE[k] = type(_ops.TUNE[k])(float(v))
-    if args.workload in ("barovik", "navalorn", "nuzinex", "torutar", "vavupel"):
+    if args.workload in ("barovik", "navalorn", "nuzinex", "torutar", "vavupel", "sofopel"):
         return measure_hybrid(args)
     if args.workload != "8b":
         return run_workload(args.workload, args)
