@@ -610,10 +610,10 @@ int gi_linear_state_rot(float* o, const void* q, long ldq, const void* k, long l
                         int n_tokens, void* stream);
 
 // ---- a stream joined once a layer; heads that are the difference of two maps; decays per key channel ------------------------
-// x += scale * y (float32 rows of d numbers side by side; `settle`: partial sums pending for y), y = 0, and, unless h is null,
+// x += scale * y (float32 rows of d numbers side by side; `first`, `second`: partial sums of up to two products pending for y), y = 0, and, unless h is null,
 // h = x / sqrt(mean(x^2) + eps) * w in h_dtype.
 int gi_join_rows(float* x, float* y, float scale, void* h, int h_dtype, const void* w, int w_dtype, int n_rows, int d, float eps,
-                 gi_settle_t settle, void* stream);
+                 gi_settle_t first, gi_settle_t second, void* stream);
 // Float32 rows [q: heads x 2 x n | k: kv_heads x 2 x n | v: kv_heads x m] through a causal convolution (conv [taps][channels], or
 // taps 0; older inputs in `state`, (taps - 1) * channels floats a slot, oldest first), maps of q and k turned by `table`
 // ([tokens][half] (cos, sin)); q: rows [heads][2][2n], each map's query with zeros in the other's place; keys (both maps side by

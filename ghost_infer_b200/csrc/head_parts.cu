@@ -95,6 +95,117 @@ head_prepare_kernel(T* __restrict__ q_out, long ldq, const float* in, long ld, c
   }
 }
 
+// The same where heads, the rotated part and the rows come in whole groups of four: a warp takes one head of one token, its lanes
+// four neighbouring numbers at a time (NV groups), kept in registers; pairs half the rotated width apart meet in shared memory.
+template <typename T, typename TW, int NV>
+__global__ void __launch_bounds__(256)
+head_prepare_warp_kernel(T* __restrict__ q_out, long ldq, const float* in, long ld, const TW* __restrict__ bq, const TW* __restrict__ bk,
+                         const TW* __restrict__ bv, const TW* __restrict__ wq, const TW* __restrict__ wk, int norm_q, int norm_k, int norm_v,
+                         float eps, const float2* table, int half, int adjacent, const int* positions, const int* slots,
+                         const int* block_table, int max_pages, T* kcache, T* vcache, int n_heads, int n_kv, int hd, int hdv, unsigned total) {
+  __shared__ float4 turn[8][32 * NV];
+  gi::pdl_prologue();
+  const unsigned item = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (item >= total) return;
+  const int lane = threadIdx.x & 31;
+  const unsigned heads = n_heads + 2 * n_kv, t = item / heads;
+  const int hh = (int)(item - t * heads);
+  const bool is_q = hh < n_heads, is_k = !is_q && hh < n_heads + n_kv;
+  const int g = is_q ? hh : (is_k ? hh - n_heads : hh - n_heads - n_kv);       // the head among its kind
+  const int n = (is_q || is_k) ? hd : hdv;
+  const int c0 = is_q ? g * hd : (is_k ? (n_heads + g) * hd : (n_heads + n_kv) * hd + g * hdv);
+  const float* r = in + (size_t)t * ld + c0;
+  const TW* b = is_q ? bq : (is_k ? bk : bv);
+  const TW* w = is_q ? wq : (is_k ? wk : nullptr);
+  const bool norm = is_q ? norm_q : (is_k ? norm_k : norm_v);
+  float4 v[NV];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = lane * 4 + 128 * j;
+    v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < n) {
+      v[j] = gi::ld4(r + i);
+      if (b != nullptr) {
+        const TW* bb = b + (size_t)g * n + i;
+        v[j].x += gi::ldf(bb); v[j].y += gi::ldf(bb + 1); v[j].z += gi::ldf(bb + 2); v[j].w += gi::ldf(bb + 3);
+      }
+      v[j] = make_float4(rounded<T>(v[j].x), rounded<T>(v[j].y), rounded<T>(v[j].z), rounded<T>(v[j].w));
+    }
+    ss = fmaf(v[j].x, v[j].x, ss); ss = fmaf(v[j].y, v[j].y, ss); ss = fmaf(v[j].z, v[j].z, ss); ss = fmaf(v[j].w, v[j].w, ss);
+  }
+  if (norm) {
+    const float rs = 1.0f / sqrtf(gi::warp_sum(ss) / (float)n + eps);
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int i = lane * 4 + 128 * j;
+      if (i >= n) continue;
+      v[j].x *= rs; v[j].y *= rs; v[j].z *= rs; v[j].w *= rs;
+      if (w != nullptr) { v[j].x *= gi::ldf(w + i); v[j].y *= gi::ldf(w + i + 1); v[j].z *= gi::ldf(w + i + 2); v[j].w *= gi::ldf(w + i + 3); }
+    }
+  }
+  const int rot = (is_q || is_k) ? 2 * half : 0;
+  if (rot > 0) {
+    const float2* cs = table + (size_t)t * half;
+    if (adjacent) {
+#pragma unroll
+      for (int j = 0; j < NV; ++j) {
+        const int i = lane * 4 + 128 * j;
+        float ra, rb;
+        if (i < rot) { gi::rotate_pair(v[j].x, v[j].y, cs[i >> 1], &ra, &rb); v[j].x = ra; v[j].y = rb; }
+        if (i + 2 < rot) { gi::rotate_pair(v[j].z, v[j].w, cs[(i >> 1) + 1], &ra, &rb); v[j].z = ra; v[j].w = rb; }
+      }
+    } else {
+      float4* mine = turn[threadIdx.x >> 5];
+#pragma unroll
+      for (int j = 0; j < NV; ++j) mine[lane + 32 * j] = v[j];
+      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < NV; ++j) {
+        const int i = lane * 4 + 128 * j;
+        if (i >= rot) continue;
+        const bool first = i < half;
+        const int p = first ? i : i - half;                       // the pair of the group's first number
+        const float4 o = mine[(first ? i + half : p) / 4];
+        const float4 c01 = *reinterpret_cast<const float4*>(cs + p), c23 = *reinterpret_cast<const float4*>(cs + p + 2);
+        const float2 c[4] = {make_float2(c01.x, c01.y), make_float2(c01.z, c01.w), make_float2(c23.x, c23.y), make_float2(c23.z, c23.w)};
+        const float a[4] = {first ? v[j].x : o.x, first ? v[j].y : o.y, first ? v[j].z : o.z, first ? v[j].w : o.w};
+        const float e[4] = {first ? o.x : v[j].x, first ? o.y : v[j].y, first ? o.z : v[j].z, first ? o.w : v[j].w};
+        float ra[4], rb[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) gi::rotate_pair(a[k], e[k], c[k], &ra[k], &rb[k]);
+        v[j] = first ? make_float4(ra[0], ra[1], ra[2], ra[3]) : make_float4(rb[0], rb[1], rb[2], rb[3]);
+      }
+    }
+  }
+  T* out;
+  if (is_q) {
+    out = q_out + (size_t)t * ldq + c0;
+  } else {
+    const int slot = slots[t], pos = max(positions[t], 0);
+    const int page = slot >= 0 ? block_table[(size_t)slot * max_pages + pos / PAGE_TOKENS] : 0;
+    out = (is_k ? kcache : vcache) + (((size_t)page * n_kv + g) * PAGE_TOKENS + pos % PAGE_TOKENS) * n;
+  }
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = lane * 4 + 128 * j;
+    if (i < n) gi::st4(out + i, v[j]);
+  }
+}
+
+// Heads of whole groups of four: a thread takes four neighbouring numbers.
+template <typename T>
+__global__ void __launch_bounds__(256)
+head_gate4_kernel(T* __restrict__ out, const T* a, const float* g, long ldg, unsigned n_heads, unsigned hdv, unsigned total) {
+  gi::pdl_prologue();
+  const unsigned i = blockIdx.x * 256 + threadIdx.x;
+  if (i >= total) return;
+  const unsigned per = hdv / 4, head = i / per, t = head / n_heads, h = head - t * n_heads;
+  const float s = sigmoid_f(g[(size_t)t * ldg + h]);
+  const float4 v = gi::ld4(a + (size_t)i * 4);
+  gi::st4(out + (size_t)i * 4, make_float4(v.x * s, v.y * s, v.z * s, v.w * s));
+}
+
 template <typename T>
 __global__ void head_gate_kernel(T* __restrict__ out, const T* a, const float* g, long ldg, int n_heads, int hdv, size_t total) {
   gi::pdl_prologue();
@@ -158,6 +269,20 @@ extern "C" int gi_head_prepare(void* q_out, long ldq, int dtype, const float* in
   if (adjacent && (hd & 1) && half > 0) return gi::fail(GI_ERR_ARG, "head_prepare: neighbouring pairs need an even head size");
   if (half > 0 && table == nullptr) return gi::fail(GI_ERR_ARG, "head_prepare: rotation without a table of angles");
   if (n_kv > 0 && (!kcache || !vcache || !block_table)) return gi::fail(GI_ERR_ARG, "head_prepare: keys and values without a cache");
+  const size_t wide = dtype == GI_BF16 ? 8 : 16;      // bytes of four numbers as stored
+  const size_t items = (size_t)n_tokens * (n_heads + 2 * (size_t)n_kv);
+  const int widest = hd > hdv ? hd : hdv;
+  if (hd % 4 == 0 && hdv % 4 == 0 && half % (adjacent ? 1 : 4) == 0 && widest <= 256 && ld % 4 == 0 && ldq % 4 == 0 && items < 0x7fffff00ul &&
+      (((uintptr_t)in | (uintptr_t)table) & 15) == 0 && (((uintptr_t)q_out | (uintptr_t)kcache | (uintptr_t)vcache) & (wide - 1)) == 0) {
+    cudaError_t e = cudaSuccess;
+    GI_DISPATCH_DTYPE(dtype, T, GI_DISPATCH_DTYPE(w_dtype, TW, {
+      auto kern = widest <= 128 ? head_prepare_warp_kernel<T, TW, 1> : head_prepare_warp_kernel<T, TW, 2>;
+      e = gi::launch(kern, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, (T*)q_out, ldq, in, ld, (const TW*)bq,
+                     (const TW*)bk, (const TW*)bv, (const TW*)wq, (const TW*)wk, norm_q, norm_k, norm_v, eps, (const float2*)table, half,
+                     adjacent, positions, slots, block_table, max_pages, (T*)kcache, (T*)vcache, n_heads, n_kv, hd, hdv, (unsigned)items);
+    }));
+    return gi::check(e, "head_prepare");
+  }
   const size_t smem = ((size_t)(n_heads + n_kv) * hd + (size_t)n_kv * hdv) * sizeof(float);
   if (smem > 160 * 1024) return gi::fail(GI_ERR_UNSUPPORTED, "head_prepare: rows of %zu bytes do not fit shared memory", smem);
   cudaError_t e = cudaSuccess;
@@ -179,6 +304,12 @@ extern "C" int gi_head_gate(void* out, const void* a, int dtype, const float* g,
   if (n_heads <= 0 || hdv <= 0) return gi::fail(GI_ERR_ARG, "head_gate: bad sizes");
   const size_t total = (size_t)n_rows * n_heads * hdv;
   cudaError_t e = cudaSuccess;
+  if (hdv % 4 == 0 && total / 4 < 0x7fffff00ul && (((uintptr_t)out | (uintptr_t)a) & 15) == 0) {
+    GI_DISPATCH_DTYPE(dtype, T,
+        e = gi::launch(head_gate4_kernel<T>, dim3(blocks_of(total / 4)), dim3(256), 0, (cudaStream_t)stream, (T*)out, (const T*)a, g, ldg,
+                       (unsigned)n_heads, (unsigned)hdv, (unsigned)(total / 4)));
+    return gi::check(e, "head_gate");
+  }
   GI_DISPATCH_DTYPE(dtype, T,
       e = gi::launch(head_gate_kernel<T>, dim3(blocks_of(total)), dim3(256), 0, (cudaStream_t)stream, (T*)out, (const T*)a, g, ldg, n_heads,
                      hdv, total));

@@ -9,37 +9,51 @@ namespace {
 
 constexpr int KD_TOK = 8;      // tokens per block
 constexpr int KD_RANK = 64;    // numbers of a row in shared memory at a time
+constexpr int KD_AHEAD = 16;   // numbers of a column of the matrix asked for at the start
+static_assert(KD_TOK == 8 && KD_AHEAD <= KD_RANK, "a row of the buffer is two groups of four tokens");
 
-// grid (token tiles, channel tiles of 256): a thread takes one channel of eight tokens
-template <typename T>
-__global__ void __launch_bounds__(256)
+// grid (token tiles, channel tiles): a thread takes one channel of eight tokens
+template <typename T, int THREADS>
+__global__ void __launch_bounds__(THREADS)
 key_decays_kernel(float* __restrict__ g, const T* low, long ldl, const float* __restrict__ up, const float* __restrict__ b, int n_tokens,
                   int rank, int channels, float inv_tau) {
-  __shared__ float sl[KD_TOK][KD_RANK];
-  gi::pdl_prologue();
+  __shared__ __align__(16) float sl[KD_RANK][KD_TOK];
+  gi::pdl_launch_dependents();
   const int t0 = blockIdx.x * KD_TOK, n = min(KD_TOK, n_tokens - t0);
-  const int c = blockIdx.y * 256 + threadIdx.x;
+  const int c = blockIdx.y * THREADS + threadIdx.x;
+  const bool live = c < channels;
+  // the matrix and the bias are written by no kernel: their first numbers are asked for before the dependency wait
+  float u[KD_AHEAD];
+#pragma unroll
+  for (int r = 0; r < KD_AHEAD; ++r) u[r] = (live && r < rank) ? up[(size_t)r * channels + c] : 0.f;
+  const float bias = live ? b[c] : 0.f;
+  gi::pdl_wait();
   float z[KD_TOK];
-  const float bias = c < channels ? b[c] : 0.f;
 #pragma unroll
   for (int t = 0; t < KD_TOK; ++t) z[t] = bias;
+  auto add = [&](int r, float w) {
+    const float4 x = *reinterpret_cast<const float4*>(&sl[r][0]), y = *reinterpret_cast<const float4*>(&sl[r][4]);
+    z[0] = fmaf(x.x, w, z[0]); z[1] = fmaf(x.y, w, z[1]); z[2] = fmaf(x.z, w, z[2]); z[3] = fmaf(x.w, w, z[3]);
+    z[4] = fmaf(y.x, w, z[4]); z[5] = fmaf(y.y, w, z[5]); z[6] = fmaf(y.z, w, z[6]); z[7] = fmaf(y.w, w, z[7]);
+  };
   for (int r0 = 0; r0 < rank; r0 += KD_RANK) {
-    const int nr = min(KD_RANK, rank - r0);
+    const int nr = min(KD_RANK, rank - r0), padded = max(nr, KD_AHEAD);
     __syncthreads();
-    for (int i = threadIdx.x; i < KD_TOK * KD_RANK; i += 256) {
-      const int t = i / KD_RANK, r = i % KD_RANK;
-      sl[t][r] = (t < n && r < nr) ? gi::ldf(low + (size_t)(t0 + t) * ldl + r0 + r) : 0.f;
+    for (int i = threadIdx.x; i < KD_TOK * padded; i += THREADS) {
+      const int t = i / padded, r = i - t * padded;
+      sl[r][t] = (t < n && r < nr) ? gi::ldf(low + (size_t)(t0 + t) * ldl + r0 + r) : 0.f;
     }
     __syncthreads();
-    if (c < channels) {
-      for (int r = 0; r < nr; ++r) {
-        const float u = up[(size_t)(r0 + r) * channels + c];
+    if (!live) continue;
+    int r = 0;
+    if (r0 == 0) {
 #pragma unroll
-        for (int t = 0; t < KD_TOK; ++t) z[t] = fmaf(sl[t][r], u, z[t]);
-      }
+      for (int k = 0; k < KD_AHEAD; ++k) add(k, u[k]);      // past the rank: zeros on both sides
+      r = KD_AHEAD;
     }
+    for (; r < nr; ++r) add(r, up[(size_t)(r0 + r) * channels + c]);
   }
-  if (c >= channels) return;
+  if (!live) return;
 #pragma unroll
   for (int t = 0; t < KD_TOK; ++t)
     if (t < n) g[(size_t)(t0 + t) * channels + c] = expf(-inv_tau * ls_softplus(-z[t]));      // sigmoid(z) = exp(-softplus(-z))
@@ -52,11 +66,15 @@ extern "C" int gi_key_decays(float* g, const void* low, long ldl, int dtype, con
   if (n_tokens <= 0) return GI_OK;
   if (rank <= 0 || channels <= 0 || !(tau > 0.f)) return gi::fail(GI_ERR_ARG, "key_decays: bad sizes (rank %d, channels %d, tau %g)", rank, channels, tau);
   if (!g || !low || !up || !b) return gi::fail(GI_ERR_ARG, "key_decays: a missing pointer");
-  const dim3 grid((n_tokens + KD_TOK - 1) / KD_TOK, (channels + 255) / 256);
+  // few tokens: narrower blocks, so that more SMs take part
+  const bool few = n_tokens <= 64;
+  const int threads = few ? 64 : 256;
+  const dim3 grid((n_tokens + KD_TOK - 1) / KD_TOK, (channels + threads - 1) / threads);
   if (grid.y > 65535) return gi::fail(GI_ERR_UNSUPPORTED, "key_decays: too many channels");
   cudaError_t e = cudaSuccess;
   GI_DISPATCH_DTYPE(dtype, T,
-      e = gi::launch(key_decays_kernel<T>, grid, dim3(256), 0, (cudaStream_t)stream, g, (const T*)low, ldl, up, b, n_tokens, rank, channels, 1.0f / tau));
+      e = few ? gi::launch(key_decays_kernel<T, 64>, grid, dim3(threads), 0, (cudaStream_t)stream, g, (const T*)low, ldl, up, b, n_tokens, rank, channels, 1.0f / tau)
+              : gi::launch(key_decays_kernel<T, 256>, grid, dim3(threads), 0, (cudaStream_t)stream, g, (const T*)low, ldl, up, b, n_tokens, rank, channels, 1.0f / tau));
   return gi::check(e, "key_decays");
 }
 

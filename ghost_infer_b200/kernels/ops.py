@@ -142,7 +142,7 @@ def _bind():
         "gi_latent_prepare_q": [P, P, I, L, P, P, I, F, P, I, P, P, P, I, P, I, I, I, I, I, P, L, P, L, I, I, P],
         "gi_attn_latent_tc_ex": [P, L, P, P, P, L, P, P, I, P, P, P, P, I, I, I, I, I, F, I, I, I, P, P, L, P],
         "gi_linear_state_rot": [P, P, L, P, L, P, L, I, P, P, I, I, F, P, L, I, P, P, I, I, I, I, I, P],
-        "gi_join_rows": [P, P, F, P, I, P, I, I, I, F, SettleT, P],
+        "gi_join_rows": [P, P, F, P, I, P, I, I, I, F, SettleT, SettleT, P],
         "gi_map_prepare": [P, L, I, P, L, P, I, P, L, I, I, P, I, I, P, P, P, I, P, P, I, I, I, I, I, P],
         "gi_map_difference": [P, P, I, I, I, I, F, F, F, P],
         "gi_key_decays": [P, P, L, I, P, P, I, I, I, F, P],
@@ -367,27 +367,43 @@ def as_carrier(t: torch.Tensor) -> torch.Tensor:
     return t if type(t) is Carrier else t.as_subclass(Carrier)
 
 
-_pending_scratch: Dict[int, torch.Tensor] = {}
+_pending_scratch: Dict[tuple, torch.Tensor] = {}       # (device, 0 or 1: the first or second product into a stream, 2: a stored product) -> scratch
 _defer_target: Optional[torch.Tensor] = None
+_defer_two = False
 
 
 def _take_pending(x: torch.Tensor):
+    """The sums of one product that are pending for `x` (a second product's, if any, are settled first)."""
     if type(x) is not Carrier:
         return None
-    return x.__dict__.pop("_gi_pending", None)
+    second = x.__dict__.pop("_gi_pending2", None)
+    first = x.__dict__.pop("_gi_pending", None)
+    if second is not None:
+        lib = _bind()
+        _check(lib, lib.gi_settle(x.data_ptr(), second[0], None, x.shape[0], x.shape[1], _stream()))
+    return first
+
+
+def _take_two_pending(x: torch.Tensor):
+    """The sums of up to two products that are pending for `x`."""
+    if type(x) is not Carrier:
+        return None, None
+    return x.__dict__.pop("_gi_pending", None), x.__dict__.pop("_gi_pending2", None)
 
 
 @contextlib.contextmanager
-def defer_into(x: torch.Tensor):
+def defer_into(x: torch.Tensor, two: bool = False):
     """Inside, a product accumulated into `x` (this very object, a `Carrier`) may leave partial sums pending.
-    Whoever reads `x` next settles them: `rmsnorm` while it reads the rows, anything else through `settle`."""
-    global _defer_target
-    prev = _defer_target
+    Whoever reads `x` next settles them: `rmsnorm` while it reads the rows, anything else through `settle`.
+    `two`: a second product may leave its own as well (`join_rows` reads both; for other readers they are added first)."""
+    global _defer_target, _defer_two
+    prev = _defer_target, _defer_two
     _defer_target = x if (TUNE["defer_residual"] and type(x) is Carrier and x.is_cuda) else None
+    _defer_two = bool(two)
     try:
         yield
     finally:
-        _defer_target = prev
+        _defer_target, _defer_two = prev
 
 
 _defer_store = False
@@ -424,18 +440,19 @@ def settle(x: torch.Tensor) -> None:
 
 def drop_pending(x: torch.Tensor) -> None:
     """Forgets partial sums pending for `x` (the stream is not read again)."""
-    _take_pending(x)
+    _take_two_pending(x)
 
 
 def _defer_ok(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> bool:
     return (_defer_target is not None and out is _defer_target and out.dtype == torch.float32
             and out.is_contiguous() and out.shape[1] % 4 == 0 and out.shape[1] <= 8192 and out.data_ptr() % 16 == 0
-            and not has_pending(out))
+            and (not has_pending(out) or (_defer_two and "_gi_pending2" not in out.__dict__ and not out.__dict__["_gi_pending"][1])))
 
 
 def _gemm_stream_deferred(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int = 4) -> torch.Tensor:
     lib = _bind()
-    key = a.device.index if a.device.index is not None else torch.cuda.current_device()
+    second = mode != SKINNY_STORE_DEFER and has_pending(out)
+    key = (a.device.index if a.device.index is not None else torch.cuda.current_device(), 2 if mode == SKINNY_STORE_DEFER else int(second))
     if key not in _pending_scratch:
         _pending_scratch[key] = torch.empty(int(lib.gi_gemm_stream_scratch_floats()), dtype=torch.float32, device=a.device)
     scratch = _pending_scratch[key]
@@ -448,7 +465,7 @@ def _gemm_stream_deferred(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, m
     n_ctas, kb, nt = c_int(0), c_int(0), c_int(0)
     lib.gi_gemm_stream_geometry(m, n, k, ctypes.byref(n_ctas), ctypes.byref(kb), ctypes.byref(nt))
     tabs = _settle_tables(a.device, (n + 127) // 128, kb.value, n_ctas.value)
-    out.__dict__["_gi_pending"] = (SettleT(scratch.data_ptr(), tabs[0].data_ptr(), tabs[1].data_ptr(), tabs[2].data_ptr(), nt.value),
+    out.__dict__["_gi_pending2" if second else "_gi_pending"] = (SettleT(scratch.data_ptr(), tabs[0].data_ptr(), tabs[1].data_ptr(), tabs[2].data_ptr(), nt.value),
                                    mode == SKINNY_STORE_DEFER)
     return out
 
@@ -2574,7 +2591,7 @@ def linear_state_rot(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: t
 # ---- a stream joined once a layer, heads that are the difference of two maps, decays per key channel ------------------------
 def join_rows(x: torch.Tensor, y: torch.Tensor, scale: float, read=None) -> Optional[torch.Tensor]:
     """x += scale * y (float32 rows), y zeroed; returns, where `read` (weight, eps, dtype) is given, the rows' RMS norm.  Partial
-    sums that a deferred product left for y are added on the way."""
+    sums that up to two deferred products left for y are added on the way."""
     lib = _bind()
     settle(x)
     for t, what in ((x, "stream rows"), (y, "sublayer rows")):
@@ -2589,17 +2606,17 @@ def join_rows(x: torch.Tensor, y: torch.Tensor, scale: float, read=None) -> Opti
         if w.numel() != d or not w.is_contiguous():
             raise KernelError(f"the norm's weight has {w.numel()} values, the rows are {d} wide")
         h = torch.empty((n, d), dtype=dtype, device=x.device)
-    rec = SettleT(None, None, None, None, 0)
+    recs = [SettleT(None, None, None, None, 0)] * 2
     if has_pending(y):
         threads = 1024 if d >= 4096 else (512 if d >= 2048 else 256)
         aligned = all(t is None or t.data_ptr() % 16 == 0 for t in (x, y, w))
         if y.__dict__["_gi_pending"][1] or d % 4 or d > 16 * threads or not aligned:
             settle(y)
         else:
-            rec = _take_pending(y)[0]
+            recs = [r[0] if r is not None else e for r, e in zip(_take_two_pending(y), recs)]
     _check(lib, lib.gi_join_rows(x.data_ptr(), y.data_ptr(), float(scale), h.data_ptr() if h is not None else None,
                                  _dt(h, "normed rows") if h is not None else F32, w.data_ptr() if w is not None else None,
-                                 _dt(w, "norm weight") if w is not None else F32, n, d, float(eps), rec, _stream()))
+                                 _dt(w, "norm weight") if w is not None else F32, n, d, float(eps), recs[0], recs[1], _stream()))
     return h
 
 

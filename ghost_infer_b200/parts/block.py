@@ -101,7 +101,7 @@ class SandwichResidual(Block):
 @register("block", "parallel_residual")
 class ParallelResidual(Block):
     """x += s * (mixer(n(x)) + ffn(n(x))), s = `params["scale"]` (1 unless given): one norm, which both sublayers read.  They add
-    into 32-bit rows of their own; one pass joins those to the stream (with whatever partial sums the last product left in them),
+    into 32-bit rows of their own; one pass joins those to the stream (with whatever partial sums the two last products left in them),
     zeroes them for the next layer and, where the next reader of the stream is a norm that says so (`row_read`), does that norm
     on the way.  Stream, norms and sums are 32-bit."""
 
@@ -119,11 +119,9 @@ class ParallelResidual(Block):
         runs = [lambda: self.mixer.forward(h, y, step, memory)] if self.mixer is not None else []
         if self.ffn is not None:
             runs.append(lambda: self.ffn.forward(h, y, step))
-        for run in runs[:-1]:
-            run()
-        if runs:
-            with ops.defer_into(y):       # nothing but the join reads the rows after the last product
-                runs[-1]()
+        with ops.defer_into(y, two=True):      # nothing but the join reads the rows: both last products may leave it their sums
+            for run in runs:
+                run()
         reader = step.next_reader
         read = reader.row_read(step) if reader is not None and hasattr(reader, "row_read") else None
         with ops.bucket("norm"):

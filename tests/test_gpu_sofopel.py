@@ -254,6 +254,44 @@ def test_joining_rows_with_partial_sums(m, width, normed):
         torch.testing.assert_close(h.double(), want / torch.sqrt((want ** 2).mean(-1, keepdim=True) + 1e-5) * nw.double(), rtol=2e-5, atol=2e-5)
 
 
+@pytest.mark.parametrize("m,width", [(1, 4096), (16, 2048), (3, 1536), (8, 8192)])
+def test_partial_sums_of_two_products(m, width):
+    """Two products into the same rows leave their cut tiles pending side by side: the join adds both, as does anyone else who reads
+    the rows; a product stored for another reader in between does not disturb them."""
+    from ghost_infer_b200.kernels import ops
+    g = torch.Generator(device="cuda:0").manual_seed(m + width)
+    rnd = lambda *s: torch.randn(s, device="cuda:0", generator=g)
+    k1, k2 = 1024, 1536
+    a1, a2 = rnd(m, k1).bfloat16(), rnd(m, k2).bfloat16()
+    w1, w2 = (rnd(width, k1) / k1 ** 0.5).bfloat16(), (rnd(width, k2) / k2 ** 0.5).bfloat16()
+    x, y0 = rnd(m, width), rnd(m, width)
+    total = y0.double() + a1.double() @ w1.double().T + a2.double() @ w2.double().T
+    for how in ("join", "settle", "torch", "third", "norm"):
+        y = ops.as_carrier(y0.clone())
+        with ops.defer_into(y, two=True):
+            ops.linear(a1, w1, out=y, accumulate=True)
+            with ops.defer_store():
+                ops.linear(a2, w2, out_dtype=torch.bfloat16)
+            ops.linear(a2, w2, out=y, accumulate=True)
+            if how == "third":
+                ops.linear(a1, w1, out=y, accumulate=True)
+        if how == "join":
+            x1 = ops.as_carrier(x.clone())
+            ops.join_rows(x1, y, 0.7)
+            torch.testing.assert_close(x1.as_subclass(torch.Tensor).double(), x.double() + 0.7 * total, rtol=1e-5, atol=3e-5)
+            assert float(y.as_subclass(torch.Tensor).abs().max()) == 0.0
+        elif how == "norm":
+            h = ops.rmsnorm(y, torch.ones((width,), device="cuda:0"), 1e-5, torch.float32)
+            torch.testing.assert_close(h.double(), total / torch.sqrt((total ** 2).mean(-1, keepdim=True) + 1e-5), rtol=2e-5, atol=2e-5)
+        else:
+            got = (y + 0.0) if how == "torch" else y
+            if how != "torch":
+                ops.settle(y)
+            want = total + (a1.double() @ w1.double().T if how == "third" else 0.0)
+            torch.testing.assert_close(got.as_subclass(torch.Tensor).double(), want, rtol=1e-5, atol=3e-5)
+        assert not ops.has_pending(y) and "_gi_pending2" not in y.__dict__
+
+
 @pytest.mark.parametrize("heads,kv,dim,vdim,taps,rot,adjacent", [(4, 2, 16, 24, 4, 8, True), (2, 1, 64, 128, 4, 64, True), (3, 3, 8, 12, 3, 6, True),
                                                                  (3, 1, 6, 5, 2, 2, True), (2, 2, 7, 9, 6, 6, True), (4, 2, 12, 8, 2, 12, False),
                                                                  (1, 1, 4, 4, 1, 0, True), (5, 5, 8, 4, 0, 4, True)])
