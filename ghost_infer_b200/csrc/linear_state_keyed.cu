@@ -12,6 +12,17 @@ constexpr int KD_RANK = 64;    // numbers of a row in shared memory at a time
 constexpr int KD_AHEAD = 16;   // numbers of a column of the matrix asked for at the start
 static_assert(KD_TOK == 8 && KD_AHEAD <= KD_RANK, "a row of the buffer is two groups of four tokens");
 
+// sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau).  The 16-bit path takes exponential and logarithm by the approximate instructions
+// and log(1 + e) for small e by its series, so that softplus stays within about 1e-7, which is all a decay near 1 can feel.
+template <bool QUICK>
+__device__ __forceinline__ float kd_decay(float z, float inv_tau) {
+  if (!QUICK) return expf(-inv_tau * ls_softplus(-z));
+  const float e = __expf(-z);
+  const float small = e * fmaf(e, fmaf(e, 1.0f / 3.0f, -0.5f), 1.0f);
+  const float sp = z < -20.f ? -z : (e < 0.005f ? small : __logf(1.0f + e));
+  return __expf(-inv_tau * sp);
+}
+
 // grid (token tiles, channel tiles): a thread takes one channel of eight tokens
 template <typename T, int THREADS>
 __global__ void __launch_bounds__(THREADS)
@@ -56,7 +67,7 @@ key_decays_kernel(float* __restrict__ g, const T* low, long ldl, const float* __
   if (!live) return;
 #pragma unroll
   for (int t = 0; t < KD_TOK; ++t)
-    if (t < n) g[(size_t)(t0 + t) * channels + c] = expf(-inv_tau * ls_softplus(-z[t]));      // sigmoid(z) = exp(-softplus(-z))
+    if (t < n) g[(size_t)(t0 + t) * channels + c] = kd_decay<sizeof(T) == 2>(z[t], inv_tau);
 }
 
 }  // namespace
