@@ -381,7 +381,7 @@ def test_decays_per_key(rows, rank, channels, tau):
         torch.testing.assert_close(ops.key_decays(x, up, b, tau).double(), want, rtol=2e-5, atol=1e-30)
 
 
-@pytest.mark.parametrize("K,V,heads", [(16, 24, 2), (48, 64, 3), (5, 7, 1), (64, 130, 2), (128, 64, 2), (200, 40, 1), (256, 8, 1), (6, 3, 5), (30, 33, 2)])
+@pytest.mark.parametrize("K,V,heads", [(16, 24, 2), (40, 56, 3), (5, 7, 1), (64, 130, 2), (128, 64, 2), (200, 40, 1), (256, 8, 1), (6, 3, 5), (30, 33, 2)])
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_recurrence_with_decays_per_key(K, V, heads, dtype):
     """Sequences in portions, among others one token each (the other instance of the kernel), with decays from 0 to 1; the state
